@@ -96,7 +96,8 @@ enum {
     SMELT_CONST_SKIP_UNLESS_POS1_LT = 10,
     SMELT_CONST_SKIP_UNLESS_POS1_GE = 11,
     SMELT_CONST_CACHE_SEQ_CAPACITY = 12,
-    SMELT_CONST_SKIP_UNLESS_SEQ_LEN_LT = 13 /* prompt chunks only: the dispatch runs only while seqLen < value */
+    SMELT_CONST_SKIP_UNLESS_SEQ_LEN_LT = 13, /* prompt chunks only: the dispatch runs only while seqLen < value */
+    SMELT_CONST_LOGIT_ROWS = 14 /* prompt chunks only (no reference counterpart): how many rows of the chunk want logits; the dispatch is skipped when none does */
 };
 enum { SMELT_OP_DISPATCH = 0, SMELT_OP_SWAP = 1 };
 enum { SMELT_SLOT_CUR = -1, SMELT_SLOT_ALT = -2 };
@@ -178,6 +179,12 @@ SMELT_CUDA_API int smelt_cuda_pipeline_supported(const char* name);
  * start_pos + seq_len must stay inside min(context_limit, cache_seq_capacity). */
 SMELT_CUDA_API smelt_status smelt_cuda_enqueue_prefill(smelt_cuda_ctx* ctx, const smelt_dispatch_record* table, size_t n_records,
                                                        const int32_t* tokens_host, int32_t seq_len, int32_t start_pos);
+/* The same with a list of the chunk's rows whose logits are asked for (ascending or not, each in [0, seq_len); n_rows may
+ * be 0).  A table that binds SMELT_CONST_LOGIT_ROWS reads the list from slot 36 and leaves n_rows rows of logits and ids;
+ * smelt_cuda_enqueue_prefill asks for the last row. */
+SMELT_CUDA_API smelt_status smelt_cuda_enqueue_prefill_rows(smelt_cuda_ctx* ctx, const smelt_dispatch_record* table, size_t n_records,
+                                                            const int32_t* tokens_host, int32_t seq_len, int32_t start_pos,
+                                                            const int32_t* rows_host, int32_t n_rows);
 SMELT_CUDA_API smelt_status smelt_cuda_decode_step(smelt_cuda_ctx* ctx, const smelt_dispatch_record* table, size_t n_records,
                                                    const int32_t* tokens, int32_t position, int32_t* out_tokens);
 /* Enqueue-only form (encodeTrunkDecode, SmeltRuntime.swift:5029-5091): no wait, no readback.
@@ -298,6 +305,46 @@ SMELT_CUDA_API smelt_status smelt_cuda_build_hybrid_prefill_table(smelt_cuda_ctx
 SMELT_CUDA_API smelt_status smelt_cuda_build_prefill_table(smelt_cuda_ctx* ctx, const smelt_decoder_desc* desc,
                                                            const smelt_layer_ref* layers, uint32_t max_chunk,
                                                            smelt_dispatch_record* records, size_t* n_records);
+
+/* ── decoders with dense 16-bit weights (no reference counterpart) ──
+ * bf16 matrices and an fp32 residual stream; parallel layers x += mixer(h) + ff(h) with h = x gain / rms(x), one gain per
+ * layer; attention without rotation over a sliding window and pooled blocks, normed queries and keys, softcapped scores
+ * and a softmax with one more in its denominator; an xIELU feed-forward (ff may be 0: none); learned positions; a range of
+ * layers that runs several times, each pass with its own cache, entered through x <- loop_in [x; embedding output].
+ * Weights image (offsets in bytes, 128-byte aligned tensors, bf16, columns zero-padded to a multiple of 64 where noted):
+ *   embedding [vocab, width], positions [max_positions, width], loop_in [width, 2 pad64(width)] (each half padded),
+ *   lm_head [vocab, pad64(width)]; per layer in_proj = rows q | k | v | up [heads dim + kv_heads (dim + vdim) + ff,
+ *   pad64(width)], out_proj = columns o | down [width, pad64(heads vdim + ff)], q_norm and k_norm [dim].
+ * precision: the type of a prompt chunk's activations and of the cache; a decode step keeps activations in fp32. */
+enum { SMELT_DENSE_BF16 = 0, SMELT_DENSE_F32 = 1 };
+typedef struct {
+    int32_t heads, kv_heads, dim, vdim;
+    uint32_t window, pool;   /* a query at i sees j > i - window, and blocks of pool positions that end at i - window or before */
+    int32_t ff;
+    float scale, softcap;    /* softcap <= 0: none */
+    float norm_gain;
+    float act_rising, act_falling; /* softplus(p), 1/2 + softplus(q) */
+    uint64_t in_proj, out_proj, q_norm, k_norm;
+} smelt_dense_layer;
+typedef struct {
+    int32_t layers, width, vocab, precision;
+    uint32_t max_positions;
+    int32_t loop_start, loop_stop, loop_times; /* layers [start, stop) run `times` times; start == stop: no loop */
+    float eps, embedding_scale, final_gain;
+    uint64_t embedding, positions, loop_in, lm_head;
+} smelt_dense_desc;
+/* Decode table (one sequence): allocates activations and one K and one V cache slot per layer run, each holding a ring of
+ * window tokens and the block means, and configures the context.  max_chunk: the longest prompt chunk the ring must take.
+ * Null ctx / records: counts only. */
+SMELT_CUDA_API smelt_status smelt_cuda_build_dense_decoder(smelt_cuda_ctx* ctx, const smelt_dense_desc* desc, const smelt_dense_layer* layers,
+                                                           uint32_t capacity, uint32_t max_chunk, smelt_dispatch_record* records, size_t* n_records);
+/* The prompt-chunk table of the same decoder (same capacity and max_chunk), for smelt_cuda_enqueue_prefill / _rows: logits
+ * fp32 in slot 16, one row per wanted row.  Build it after the decode table and before a graph. */
+SMELT_CUDA_API smelt_status smelt_cuda_build_dense_prefill_table(smelt_cuda_ctx* ctx, const smelt_dense_desc* desc, const smelt_dense_layer* layers,
+                                                                 uint32_t capacity, uint32_t max_chunk, smelt_dispatch_record* records, size_t* n_records);
+/* The cache slots of the decoder: n consecutive slots, K and V of each layer run in the order of execution.  For
+ * snapshots they are position-less state (a ring cannot be cut to a shorter length). */
+SMELT_CUDA_API smelt_status smelt_cuda_dense_cache_slots(const smelt_dense_desc* desc, int32_t* first_slot, int32_t* n_slots);
 
 /* The pipeline names of the table smelt_cuda_build_prefill_table writes, in the order of the indices a table built
  * without a context carries (0, 1, ...): newline separated, as smelt_cuda_decoder_pipelines reports the decode table's. */

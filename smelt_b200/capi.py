@@ -94,6 +94,20 @@ class DeltaRef(C.Structure):
                 ("conv_weight", C.c_uint64), ("a_log", C.c_uint64), ("dt_bias", C.c_uint64), ("norm_weight", C.c_uint64)]
 
 
+class DenseLayer(C.Structure):
+    """``smelt_dense_layer``: one layer of a decoder with dense 16-bit weights."""
+    _fields_ = [("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("window", C.c_uint32), ("pool", C.c_uint32),
+                ("ff", C.c_int32), ("scale", C.c_float), ("softcap", C.c_float), ("norm_gain", C.c_float), ("act_rising", C.c_float),
+                ("act_falling", C.c_float), ("in_proj", C.c_uint64), ("out_proj", C.c_uint64), ("q_norm", C.c_uint64), ("k_norm", C.c_uint64)]
+
+
+class DenseDesc(C.Structure):
+    """``smelt_dense_desc``."""
+    _fields_ = [("layers", C.c_int32), ("width", C.c_int32), ("vocab", C.c_int32), ("precision", C.c_int32), ("max_positions", C.c_uint32),
+                ("loop_start", C.c_int32), ("loop_stop", C.c_int32), ("loop_times", C.c_int32), ("eps", C.c_float), ("embedding_scale", C.c_float),
+                ("final_gain", C.c_float), ("embedding", C.c_uint64), ("positions", C.c_uint64), ("loop_in", C.c_uint64), ("lm_head", C.c_uint64)]
+
+
 class PackageOptions(C.Structure):
     _fields_ = [("context_capacity", C.c_uint32), ("context_limit", C.c_uint32)]
 

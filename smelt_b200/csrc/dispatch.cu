@@ -11,6 +11,7 @@
 #include <cstring>
 
 #include "affine_matvec.h"
+#include "dense.h"
 #include "glue.h"
 #include "runtime.h"
 
@@ -135,6 +136,34 @@ bool parse_pipeline(const char* entry, Pipeline* out) {
         p.kind = name == "smelt_rmsnorm_affine_qkv" ? PK_FUSED_NORM_QKV : PK_FUSED_NORM_GATEUP;
         *out = p;
         return true;
+    }
+    // Kernels of the dense-weight decoders; the typed ones end in the type of their activations and caches (bits = DenseType).
+    {
+        struct Dense { const char* name; PipeKind kind; int mode; bool typed, shaped; };
+        static const Dense dense[] = {
+            {"smelt_embed_positions", PK_EMBED_POSITIONS, 0, false, false},
+            {"smelt_dense_matvec", PK_DENSE_MATVEC, kDenseStoreF32, false, true},
+            {"smelt_dense_matvec_xielu", PK_DENSE_MATVEC, kDenseStoreF32, false, true},
+            {"smelt_dense_matvec_add", PK_DENSE_MATVEC, kDenseAddF32, false, true},
+            {"smelt_dense_gemm", PK_DENSE_GEMM, kDenseStoreF32, true, true},
+            {"smelt_dense_gemm_xielu", PK_DENSE_GEMM, kDenseStoreAct, true, true},
+            {"smelt_dense_gemm_add", PK_DENSE_GEMM, kDenseAddF32, true, true},
+            {"smelt_scalar_norm_rows", PK_SCALAR_NORM_ROWS, 0, true, false},
+            {"smelt_pair_rows", PK_PAIR_ROWS, 0, true, false},
+            {"smelt_window_append", PK_WINDOW_APPEND, 0, true, false},
+            {"smelt_window_pool", PK_WINDOW_POOL, 0, true, false},
+            {"smelt_window_attention", PK_WINDOW_ATTENTION, 0, true, true},
+            {"smelt_window_decode", PK_WINDOW_DECODE, 0, true, false},
+            {"argmax_f32_partials", PK_ARGMAX_F32_PARTIALS, 0, false, false},
+        };
+        for (const Dense& d : dense)
+            for (int t = 0; t < (d.typed ? 2 : 1); ++t)
+                if (name == (d.typed ? std::string(d.name) + (t == kDenseF32 ? "_f32" : "_bf16") : std::string(d.name))) {
+                    if (d.shaped && p.cols <= 0) return false;
+                    p.kind = d.kind; p.mode = d.mode; p.bits = t; p.fixed_shape = name == "smelt_dense_matvec_xielu" || d.mode == kDenseStoreAct;
+                    *out = p;
+                    return true;
+                }
     }
     struct Simple { const char* name; PipeKind kind; int bits; bool batched; };
     static const Simple table[] = {
@@ -379,6 +408,7 @@ struct Interp {
     int launches = 0;
     bool prefill = false;    // a prompt chunk: seq_len positions from start_pos (position == start_pos; SmeltRuntime.swift:1217-1250)
     uint32_t seq_len = 0, start_pos = 0;
+    uint32_t logit_rows = 0; // rows of the chunk whose logits are asked for
     int rope_half = 0;       // the position's cos | sin table holds this many pairs ...
     float rope_base = 0.f;   // ... for this log2(theta); 0 pairs = not written in this interpretation
 };
@@ -428,7 +458,7 @@ smelt_status resolve(Interp& in, const smelt_dispatch_record& rec, Resolved* out
             case SMELT_CONST_POSITION_PLUS1: case SMELT_CONST_CACHE_SEQ_CAPACITY:
                 break;
             case SMELT_CONST_SEQ_LEN: case SMELT_CONST_START_POS: case SMELT_CONST_START_POS_PLUS: case SMELT_CONST_SEQ_LEN_MUL:
-            case SMELT_CONST_SEQ_LEN_MOD: case SMELT_CONST_SEQ_LEN_MOD_SKIP_IF_ZERO: case SMELT_CONST_SKIP_UNLESS_SEQ_LEN_LT:
+            case SMELT_CONST_SEQ_LEN_MOD: case SMELT_CONST_SEQ_LEN_MOD_SKIP_IF_ZERO: case SMELT_CONST_SKIP_UNLESS_SEQ_LEN_LT: case SMELT_CONST_LOGIT_ROWS:
                 if (!in.prefill) return fail(ctx, SMELT_ERR_UNSUPPORTED, "record: constant kind " + std::to_string(c.kind) + " is outside the decode path");
                 break;
             default:
@@ -450,6 +480,10 @@ smelt_status resolve(Interp& in, const smelt_dispatch_record& rec, Resolved* out
                     break;
                 case SMELT_CONST_SKIP_UNLESS_SEQ_LEN_LT:
                     value = in.seq_len < c.value ? 1u : 0u; kind = SMELT_CONST_LITERAL_U32;
+                    if (value == 0) out->skip = true;
+                    break;
+                case SMELT_CONST_LOGIT_ROWS:
+                    value = in.logit_rows; kind = SMELT_CONST_LITERAL_U32;
                     if (value == 0) out->skip = true;
                     break;
                 default: break;
@@ -668,6 +702,127 @@ smelt_status run_attention(Interp& in, const Pipeline& p, const smelt_dispatch_r
     return check_cuda(ctx, launch_attention_decode(make_launch(in, r), a), p.name.c_str());
 }
 
+// Dense-weight decoders (dense_builder.cu writes these records).
+smelt_status run_dense(Interp& in, const Pipeline& p, const Resolved& r) {
+    smelt_cuda_ctx* ctx = in.ctx;
+    Launch l = make_launch(in, r);
+    const DenseType type = (DenseType)p.bits;
+    const size_t es = type == kDenseF32 ? 4 : 2;
+    auto f32 = [&](int i, float* v) { uint32_t b; const bool ok = host_u32(in, r, i, &b); if (ok) *v = as_f32(b); return ok; };
+#define NEED_F32(i, var)                                                                                  \
+    float var = 0.f;                                                                                      \
+    if (!f32(i, &var)) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, p.name + ": constant binding " #i " is missing")
+    in.launches += 1;
+    switch (p.kind) {
+        case PK_EMBED_POSITIONS: {
+            // 0 table, 1 token ids, 2 position table, 3 x, 4 copy of x; 5 width, 6 ld, 7 rows, 8 max positions, 9 scale
+            NEED_BUF(0); NEED_BUF(1); NEED_BUF(2); NEED_BUF(3); NEED_BUF(4); NEED_U32(5, width); NEED_U32(6, ld); NEED_U32(7, m); NEED_U32(8, max_pos); NEED_F32(9, scale);
+            NEED_BYTES(0, (size_t)ctx->cfg.vocab_size * width * 2); NEED_BYTES(1, (size_t)m * 4); NEED_BYTES(2, (size_t)max_pos * width * 2);
+            NEED_BYTES(3, (size_t)m * ld * 4); NEED_BYTES(4, (size_t)m * ld * 4);
+            return check_cuda(ctx, launch_embed_positions(l, (const bf16*)r.buf[0].ptr, (const int32_t*)r.buf[1].ptr, (const bf16*)r.buf[2].ptr, (float*)r.buf[3].ptr, (float*)r.buf[4].ptr,
+                                                          (int)width, (int)ld, (int)m, ctx->cfg.vocab_size, max_pos, scale), p.name.c_str());
+        }
+        case PK_DENSE_MATVEC: {
+            // name:cols:width; 0 W, 1 x, 2 second half of x (optional), 3 y, 4 y past the split (xielu); 5 rows, 6 split, 7 norm gain (optional), 8 eps, 9 rising, 10 falling
+            NEED_BUF(0); NEED_BUF(1); NEED_BUF(3); NEED_U32(5, rows);
+            DenseMatvecArgs a = {};
+            a.rows = (int)rows; a.cols = p.cols; a.width = p.group; a.out.split = (int)rows; a.ka = r.buf[2].present ? p.cols / 2 : p.cols;
+            a.w = (const bf16*)r.buf[0].ptr; a.xa = (const float*)r.buf[1].ptr; a.xb = r.buf[2].present ? (const float*)r.buf[2].ptr : nullptr;
+            a.out.y0 = r.buf[3].ptr; a.sm_count = ctx->sm_count;
+            if (p.fixed_shape) {
+                NEED_BUF(4); NEED_U32(6, split); NEED_F32(9, rising); NEED_F32(10, falling);
+                if (split > rows) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, p.name + ": split past the rows");
+                a.out.split = (int)split; a.out.rising = rising; a.out.falling = falling; a.out.y1 = r.buf[4].ptr;
+                NEED_BYTES(4, (size_t)(rows - split) * 4);
+            }
+            a.norm = f32(7, &a.gain) ? 1 : 0;
+            if (a.norm) { NEED_F32(8, eps); a.eps = eps; }
+            NEED_BYTES(0, (size_t)rows * p.cols * 2); NEED_BYTES(1, (size_t)a.ka * 4); NEED_BYTES(3, (size_t)a.out.split * 4);
+            if (a.xb) NEED_BYTES(2, (size_t)(p.cols - a.ka) * 4);
+            return check_cuda(ctx, launch_dense_matvec(l, p.mode, a), p.name.c_str());
+        }
+        case PK_DENSE_GEMM: {
+            // name:cols:width; 0 W, 1 X [m, cols], 2 y, 3 y past the split (xielu); 5 rows, 6 m, 7 split, 8 ld of y, 9 ld past the split, 10 rising, 11 falling
+            NEED_BUF(0); NEED_BUF(1); NEED_BUF(2); NEED_U32(5, rows); NEED_U32(6, m); NEED_U32(7, split); NEED_U32(8, ld0);
+            DenseGemmArgs a = {};
+            a.w = (const bf16*)r.buf[0].ptr; a.x = r.buf[1].ptr; a.rows = (int)rows; a.cols = p.cols; a.m = (int)m;
+            a.out.y0 = r.buf[2].ptr; a.out.ld0 = (int)ld0; a.out.split = (int)split;
+            if (split > rows || ld0 < split) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, p.name + ": split past the rows, or rows past the leading dimension");
+            NEED_BYTES(0, (size_t)rows * p.cols * 2); NEED_BYTES(1, (size_t)m * p.cols * es);
+            NEED_BYTES(2, ((size_t)(m - 1) * ld0 + split) * (p.mode == kDenseStoreAct ? es : 4));
+            if (p.fixed_shape) {
+                NEED_BUF(3); NEED_U32(9, ld1); NEED_F32(10, rising); NEED_F32(11, falling);
+                a.out.y1 = r.buf[3].ptr; a.out.ld1 = (int)ld1; a.out.rising = rising; a.out.falling = falling;
+                NEED_BYTES(3, ((size_t)(m - 1) * ld1 + (rows - split)) * es);
+            }
+            a.sm_count = ctx->sm_count; a.err = ctx->err_dev;
+            a.part_scratch = ctx->qmm_scratch; a.part_scratch_bytes = ctx->qmm_scratch_bytes; a.part_counters = ctx->qmm_counters;
+            return check_cuda(ctx, launch_dense_gemm(l, type, p.mode, a), p.name.c_str());
+        }
+        case PK_SCALAR_NORM_ROWS: {
+            // 0 x, 1 out, 2 row list (optional); 3 width, 4 ld, 5 m, 6 gain, 7 eps
+            NEED_BUF(0); NEED_BUF(1); NEED_U32(3, width); NEED_U32(4, ld); NEED_U32(5, m); NEED_F32(6, gain); NEED_F32(7, eps);
+            const bool list = r.buf[2].present;
+            if (list) NEED_BYTES(2, (size_t)m * 4);
+            NEED_BYTES(0, (size_t)(list ? in.seq_len : m) * ld * 4); NEED_BYTES(1, (size_t)m * ld * es);
+            return check_cuda(ctx, launch_scalar_norm_rows(l, type, (const float*)r.buf[0].ptr, list ? (const int32_t*)r.buf[2].ptr : nullptr, r.buf[1].ptr, (int)width, (int)ld, (int)m, gain, eps), p.name.c_str());
+        }
+        case PK_PAIR_ROWS: {
+            // 0 x, 1 x0, 2 out; 3 ld, 4 m
+            NEED_BUF(0); NEED_BUF(1); NEED_BUF(2); NEED_U32(3, ld); NEED_U32(4, m);
+            NEED_BYTES(0, (size_t)m * ld * 4); NEED_BYTES(1, (size_t)m * ld * 4); NEED_BYTES(2, (size_t)m * 2 * ld * es);
+            return check_cuda(ctx, launch_pair_rows(l, type, (const float*)r.buf[0].ptr, (const float*)r.buf[1].ptr, r.buf[2].ptr, (int)ld, (int)m), p.name.c_str());
+        }
+        case PK_ARGMAX_F32_PARTIALS: {
+            // 0 logits, 1 partials; 2 vocab, 3 chunk, 4 rows
+            NEED_BUF(0); NEED_BUF(1); NEED_U32(2, vocab); NEED_U32(3, chunk); NEED_U32(4, rows);
+            if (vocab == 0 || chunk == 0) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, p.name + ": vocab and chunk must be positive");
+            NEED_BYTES(0, (size_t)rows * vocab * 4); NEED_BYTES(1, (size_t)rows * ((vocab + chunk - 1) / chunk) * 8);
+            return check_cuda(ctx, launch_argmax_f32_partials(l, (const float*)r.buf[0].ptr, (uint64_t*)r.buf[1].ptr, (int)vocab, (int)chunk, (int)rows), p.name.c_str());
+        }
+        default: break;
+    }
+    // attention: 0 projections, 1 query norm, 2 key norm, 3 K cache, 4 V cache, 5 queries, 6 out;
+    // 8 heads | kv_heads << 16, 9 dim | vdim << 16, 10 window, 11 pool, 12 ring, 13 scale, 14 softcap, 15 m, 16 eps
+    NEED_BUF(3); NEED_BUF(4); NEED_U32(8, heads); NEED_U32(9, dims); NEED_U32(10, window); NEED_U32(11, pool); NEED_U32(12, ring);
+    WindowArgs a = {};
+    a.heads = heads & 0xffff; a.kv_heads = heads >> 16; a.dim = dims & 0xffff; a.vdim = dims >> 16; a.window = window; a.pool = pool; a.ring = ring;
+    if (a.heads == 0 || a.kv_heads == 0 || a.dim == 0 || a.vdim == 0 || pool == 0 || ring == 0) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, p.name + ": bad geometry");
+    a.kp = window_padded(a.dim); a.vp = window_padded(a.vdim);
+    a.blocks = ctx->cfg.cache_seq_capacity / pool;
+    a.m = 1;
+    if (p.kind != PK_WINDOW_DECODE) { NEED_U32(15, m); a.m = (int)m; }
+    const size_t rows = (size_t)a.kv_heads * (ring + a.blocks), qkv = (size_t)a.heads * a.dim + (size_t)a.kv_heads * (a.dim + a.vdim);
+    const size_t us = p.kind == PK_WINDOW_DECODE ? 4 : es;
+    NEED_BYTES(3, rows * a.kp * es); NEED_BYTES(4, rows * a.vp * es);
+    a.k_cache = r.buf[3].ptr; a.v_cache = r.buf[4].ptr;
+    a.sm_count = ctx->sm_count; a.scratch = ctx->attn_scratch; a.scratch_bytes = ctx->attn_scratch_bytes; a.counters = ctx->attn_counters;
+    if (p.kind == PK_WINDOW_POOL) return check_cuda(ctx, launch_window_pool(l, type, a), p.name.c_str());
+    NEED_BUF(5); NEED_BYTES(5, (size_t)a.m * a.heads * a.kp * us);
+    a.q = r.buf[5].ptr;
+    if (p.kind != PK_WINDOW_ATTENTION) {
+        NEED_BUF(0); NEED_BUF(1); NEED_BUF(2); NEED_F32(16, eps);
+        NEED_BYTES(0, (size_t)a.m * qkv * us); NEED_BYTES(1, (size_t)a.dim * 2); NEED_BYTES(2, (size_t)a.dim * 2);
+        a.u = r.buf[0].ptr; a.q_norm = (const bf16*)r.buf[1].ptr; a.k_norm = (const bf16*)r.buf[2].ptr; a.eps = eps;
+        if (p.kind == PK_WINDOW_APPEND) return check_cuda(ctx, launch_window_append(l, type, a), p.name.c_str());
+    }
+    NEED_BUF(6); NEED_F32(13, scale); NEED_F32(14, softcap);
+    a.z = r.buf[6].ptr; a.scale = scale; a.softcap = softcap;
+    if (p.kind == PK_WINDOW_ATTENTION) {
+        a.ldz = p.cols;
+        if (a.ldz < a.heads * a.vdim) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, p.name + ": output rows are shorter than the heads");
+        NEED_BYTES(6, ((size_t)(a.m - 1) * a.ldz + (size_t)a.heads * a.vdim) * es);
+        return check_cuda(ctx, launch_window_attention(l, type, a), p.name.c_str());
+    }
+    a.ldz = a.heads * a.vdim;
+    NEED_BYTES(6, (size_t)a.ldz * 4);
+    int launches = 1;
+    const smelt_status s = check_cuda(ctx, launch_window_decode(l, type, a, &launches), p.name.c_str());
+    in.launches += launches - 1;
+    return s;
+#undef NEED_F32
+}
+
 smelt_status run_record(Interp& in, const smelt_dispatch_record& rec_in) {
     smelt_cuda_ctx* ctx = in.ctx;
     smelt_dispatch_record rec = rec_in;
@@ -703,6 +858,9 @@ smelt_status run_record(Interp& in, const smelt_dispatch_record& rec_in) {
             return run_signed(in, p, rec, r);
         case PK_ATTN_GENERIC: case PK_ATTN_INPLACE: case PK_ATTN_ROPE: case PK_ATTN_MLX_2PASS_1:
             return run_attention(in, p, rec, r);
+        case PK_EMBED_POSITIONS: case PK_DENSE_MATVEC: case PK_DENSE_GEMM: case PK_SCALAR_NORM_ROWS: case PK_PAIR_ROWS: case PK_WINDOW_APPEND:
+        case PK_WINDOW_POOL: case PK_WINDOW_ATTENTION: case PK_WINDOW_DECODE: case PK_ARGMAX_F32_PARTIALS:
+            return run_dense(in, p, r);
         case PK_ATTN_MLX_2PASS_2: {
             // attention.metal:1146-1153: 0 partials, 1 stats, 2 out, 3 qHeads.
             NEED_BUF(0); NEED_BUF(1); NEED_BUF(2); NEED_U32(3, nq);
@@ -751,7 +909,8 @@ smelt_status run_record(Interp& in, const smelt_dispatch_record& rec_in) {
         case PK_ARGMAX_REDUCE: {
             // lut_matvec.metal:8938-8942: 0 partials, 1 out, 2 numPartials.
             NEED_BUF(0); NEED_BUF(1); NEED_U32(2, parts);
-            const int batch = batch_of(rec);
+            uint32_t rows = 0;  // 4 (extension): rows, when they are not the grid's
+            const int batch = host_u32(in, r, 4, &rows) ? (int)rows : batch_of(rec);
             NEED_BYTES(0, (size_t)parts * batch * 8); NEED_BYTES(1, (size_t)batch * 4);
             in.launches += 1;
             return check_cuda(ctx, launch_argmax_reduce(l, (const uint64_t*)r.buf[0].ptr, (int32_t*)r.buf[1].ptr, (int)parts, batch, 1), "argmax_key_reduce");
@@ -1674,7 +1833,13 @@ smelt_status smelt_cuda_enqueue_decode(smelt_cuda_ctx* ctx, const smelt_dispatch
 // SmeltRuntime.swift:1217-1250, :6160-6207).  Eager only: a prefill table's shapes change with the chunk.
 smelt_status smelt_cuda_enqueue_prefill(smelt_cuda_ctx* ctx, const smelt_dispatch_record* table, size_t n_records, const int32_t* tokens,
                                         int32_t seq_len, int32_t start_pos) {
-    if (!ctx || !table || !tokens) return SMELT_ERR_BAD_ARGUMENT;
+    const int32_t last = seq_len - 1;
+    return smelt_cuda_enqueue_prefill_rows(ctx, table, n_records, tokens, seq_len, start_pos, &last, 1);
+}
+
+smelt_status smelt_cuda_enqueue_prefill_rows(smelt_cuda_ctx* ctx, const smelt_dispatch_record* table, size_t n_records, const int32_t* tokens,
+                                             int32_t seq_len, int32_t start_pos, const int32_t* rows, int32_t n_rows) {
+    if (!ctx || !table || !tokens || n_rows < 0 || (n_rows && !rows)) return SMELT_ERR_BAD_ARGUMENT;
     if (cudaSetDevice(ctx->device) != cudaSuccess) return fail(ctx, SMELT_ERR_CUDA, "cudaSetDevice");
     if (!ctx->configured) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, "context is not configured");
     if (ctx->capturing) return fail(ctx, SMELT_ERR_UNSUPPORTED, "prefill tables are interpreted eagerly, not captured");
@@ -1686,14 +1851,26 @@ smelt_status smelt_cuda_enqueue_prefill(smelt_cuda_ctx* ctx, const smelt_dispatc
         if (tokens[i] < 0 || (uint32_t)tokens[i] >= ctx->cfg.vocab_size) return fail(ctx, SMELT_ERR_OUT_OF_RANGE, "tokenId out of range [0, " + std::to_string(ctx->cfg.vocab_size) + ")");
     Slot& ts = ctx->slots[ctx->cfg.token_id_slot];
     if (!ts.ptr || ts.bytes < (size_t)seq_len * 4) return fail(ctx, SMELT_ERR_OUT_OF_RANGE, "prefill: the token slot holds fewer than seq_len ids");
+    Slot& rs = ctx->slots[kLogitRowsSlot];  // only tables that bind it have it
+    const bool list = rs.ptr && n_rows > 0;
+    if (n_rows > seq_len || (list && (rs.bytes < (size_t)n_rows * 4 || (size_t)seq_len + n_rows > ctx->h_pinned_count - 256)))
+        return fail(ctx, SMELT_ERR_OUT_OF_RANGE, "prefill: too many logit rows");
+    for (int32_t i = 0; i < n_rows; ++i)
+        if (rows[i] < 0 || rows[i] >= seq_len) return fail(ctx, SMELT_ERR_OUT_OF_RANGE, "prefill: a logit row is outside the chunk");
     // the staging area may still feed an earlier chunk's copy
     smelt_status s = check_cuda(ctx, cudaStreamSynchronize(ctx->stream), "prefill: chunk boundary");
     if (s) return s;
     for (int32_t i = 0; i < seq_len; ++i) ctx->h_pinned[256 + i] = tokens[i];
     s = check_cuda(ctx, cudaMemcpyAsync(ts.ptr, ctx->h_pinned + 256, (size_t)seq_len * 4, cudaMemcpyHostToDevice, ctx->stream), "prefill: token ids");
     if (s) return s;
+    if (list) {
+        for (int32_t i = 0; i < n_rows; ++i) ctx->h_pinned[256 + seq_len + i] = rows[i];
+        s = check_cuda(ctx, cudaMemcpyAsync(rs.ptr, ctx->h_pinned + 256 + seq_len, (size_t)n_rows * 4, cudaMemcpyHostToDevice, ctx->stream), "prefill: logit rows");
+        if (s) return s;
+    }
     Interp in;
     in.ctx = ctx; in.device_pos = false; in.position = (uint32_t)start_pos;
+    in.logit_rows = (uint32_t)n_rows;
     in.prefill = true; in.seq_len = (uint32_t)seq_len; in.start_pos = (uint32_t)start_pos;
     in.cur = ctx->cfg.cur_slot; in.alt = ctx->cfg.alt_slot;
     for (size_t i = 0; i < n_records; ++i) {

@@ -69,7 +69,7 @@ smelt_status smelt_cuda_create(int device_ordinal, smelt_cuda_ctx** out_ctx) {
     if (!ctx) return SMELT_ERR_ALLOC;
     ctx->device = device_ordinal;
     ctx->sm_count = prop.multiProcessorCount;
-    ctx->slots.resize(256);
+    ctx->slots.resize(kSlotCount);
     bool ok = cudaStreamCreateWithFlags(&ctx->stream, cudaStreamNonBlocking) == cudaSuccess;
     ok = ok && cudaMalloc(&ctx->dyn_dev, sizeof(DynState)) == cudaSuccess;
     ok = ok && cudaMalloc(&ctx->err_dev, sizeof(uint32_t)) == cudaSuccess;

@@ -81,6 +81,16 @@ enum PipeKind : int {
     PK_DN_DELTA,
     PK_DN_FUSED_DECODE,
     PK_DN_FUSED_PREFILL,
+    PK_EMBED_POSITIONS,
+    PK_DENSE_MATVEC,
+    PK_DENSE_GEMM,
+    PK_SCALAR_NORM_ROWS,
+    PK_PAIR_ROWS,
+    PK_WINDOW_APPEND,
+    PK_WINDOW_POOL,
+    PK_WINDOW_ATTENTION,
+    PK_WINDOW_DECODE,
+    PK_ARGMAX_F32_PARTIALS,
 };
 
 struct Pipeline {
@@ -92,6 +102,7 @@ struct Pipeline {
     int bits = 0;                        // signed kernels: 1 or 2
     int planes = 0;                      // activation bit-plane kernels: planes of the view (2..6)
     int n_q = 0, n_kv = 0, head_dim = 0; // shape-specialised attention names
+    int mode = 0;                        // dense projections: DenseMode
 };
 
 // Parses a manifest pipeline entry; returns false when the kernel is not implemented.
@@ -152,6 +163,8 @@ struct smelt_cuda_ctx {
 };
 
 namespace smelt {
+constexpr int kSlotCount = 1024;
+constexpr int kLogitRowsSlot = 36;  // row list of smelt_cuda_enqueue_prefill_rows
 constexpr int kGraphBurst = 8;  // tokens per launch of the multi-token decode graph
 void destroy_decode_graphs(smelt_cuda_ctx* ctx);  // the single-token and the multi-token graph
 smelt_status fail(smelt_cuda_ctx* ctx, smelt_status code, const std::string& msg);

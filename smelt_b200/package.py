@@ -256,19 +256,24 @@ class Decoder:
         self.hybrid = hybrid
         desc.fuse_residual = int(fuse_residual)
         ctx.call("upload_weights", WEIGHTS_SLOT, image, C.c_size_t(image.nbytes))
-        n = C.c_size_t(0)
         if hybrid is not None:
-            build = lambda h, table: ctx.lib.smelt_cuda_build_hybrid_decoder(h, C.byref(desc), layers, C.byref(hybrid.desc), hybrid.refs, hybrid.kinds,
-                                                                             capacity, table, C.byref(n))
+            build = lambda h, table, n: ctx.lib.smelt_cuda_build_hybrid_decoder(h, C.byref(desc), layers, C.byref(hybrid.desc), hybrid.refs, hybrid.kinds,
+                                                                                capacity, table, n)
         else:
-            build = lambda h, table: ctx.lib.smelt_cuda_build_decoder(h, C.byref(desc), layers, capacity, batch, table, C.byref(n))
-        st = build(None, None)
-        if st != 0:
-            raise capi.SmeltError(st, "build_decoder (count) failed")
-        self.table = (capi.DispatchRecord * n.value)()
-        ctx._check(build(ctx.h, self.table))
-        self.n_records = n.value
+            build = lambda h, table, n: ctx.lib.smelt_cuda_build_decoder(h, C.byref(desc), layers, capacity, batch, table, n)
+        self.table = self._write_table(build, "build_decoder")
+        self.n_records = len(self.table)
         self.graph_ready = False
+
+    def _write_table(self, build, what: str):
+        """The records ``build(ctx or None, records or None, count)`` writes: counted first, then written."""
+        n = C.c_size_t(0)
+        st = build(None, None, C.byref(n))
+        if st != 0:
+            raise capi.SmeltError(st, f"{what} (count) failed")
+        table = (capi.DispatchRecord * n.value)()
+        self.ctx._check(build(self.ctx.h, table, C.byref(n)))
+        return table
 
     def decode_step(self, tokens, position: int) -> np.ndarray:
         tokens = np.ascontiguousarray(np.atleast_1d(tokens), dtype=np.int32)
@@ -277,8 +282,10 @@ class Decoder:
                                                            int(position), out.ctypes.data_as(C.c_void_p)))
         return out
 
-    def logits(self) -> np.ndarray:
-        out = np.empty((self.batch, self.desc.vocab), np.float16)
+    logits_dtype = np.float16
+
+    def logits(self, rows: int | None = None) -> np.ndarray:
+        out = np.empty((self.batch if rows is None else rows, self.desc.vocab), self.logits_dtype)
         self.ctx._check(self.ctx.lib.smelt_cuda_read_slot(self.ctx.h, LOGITS_SLOT, 0, out.ctypes.data_as(C.c_void_p), out.nbytes))
         return out
 
@@ -307,16 +314,13 @@ class Decoder:
     def build_prefill_table(self, max_chunk: int = 512):
         """The prompt-chunk dispatch table of this decoder in the reference's prefill record shapes
         (``smelt_cuda_build_prefill_table``); call it before ``build_graph``."""
-        n = C.c_size_t(0)
         lib, hy = self.ctx.lib, self.hybrid
         if hy is not None:
-            build = lambda h, table: lib.smelt_cuda_build_hybrid_prefill_table(h, C.byref(self.desc), self.layers, C.byref(hy.desc), hy.refs, hy.kinds,
-                                                                               int(max_chunk), table, C.byref(n))
+            build = lambda h, table, n: lib.smelt_cuda_build_hybrid_prefill_table(h, C.byref(self.desc), self.layers, C.byref(hy.desc), hy.refs, hy.kinds,
+                                                                                  int(max_chunk), table, n)
         else:
-            build = lambda h, table: lib.smelt_cuda_build_prefill_table(h, C.byref(self.desc), self.layers, int(max_chunk), table, C.byref(n))
-        self.ctx._check(build(None, None))
-        self.prefill_records = (capi.DispatchRecord * n.value)()
-        self.ctx._check(build(self.ctx.h, self.prefill_records))
+            build = lambda h, table, n: lib.smelt_cuda_build_prefill_table(h, C.byref(self.desc), self.layers, int(max_chunk), table, n)
+        self.prefill_records = self._write_table(build, "build_prefill_table")
         self.prefill_chunk = int(max_chunk)
         return self.prefill_records
 
@@ -428,6 +432,108 @@ class Decoder:
             if i + 1 < n_decode:
                 cur = self.decode_step(cur, n_prompt + i)
         return out
+
+
+class DenseDecoder(Decoder):
+    """A decoder with dense 16-bit weights (``smelt_cuda_build_dense_decoder``): one sequence, fp32 logits.
+
+    A decoded token replays the captured graph; a prompt goes through the prompt-chunk table,
+    ``max_chunk`` positions at a time.  precision: the type of a chunk's activations and of the
+    cache, "bfloat16" or "float32"."""
+
+    logits_dtype = np.float32
+    PRECISIONS = {"bfloat16": 0, "float32": 1}
+
+    def __init__(self, ctx: capi.Context, image: np.ndarray, desc: capi.DenseDesc, layers, capacity: int, precision: str = "bfloat16", max_chunk: int = 512):
+        self.ctx, self.desc, self.layers, self.capacity, self.batch, self.hybrid = ctx, desc, layers, int(capacity), 1, None
+        desc.precision = self.PRECISIONS[precision]
+        ctx.call("upload_weights", WEIGHTS_SLOT, image, C.c_size_t(image.nbytes))
+        lib = ctx.lib
+        chunk = self.prefill_chunk = int(min(max_chunk, capacity))
+        self.table = self._write_table(lambda h, t, n: lib.smelt_cuda_build_dense_decoder(h, C.byref(desc), layers, self.capacity, chunk, t, n), "build_dense_decoder")
+        self.n_records = len(self.table)
+        self.prefill_records = self._write_table(lambda h, t, n: lib.smelt_cuda_build_dense_prefill_table(h, C.byref(desc), layers, self.capacity, chunk, t, n), "build_dense_prefill_table")
+        self.graph_ready = False
+
+    def _enqueue_chunk(self, tokens, start_pos: int, rows) -> None:
+        rows = np.ascontiguousarray(rows, np.int32)
+        self.ctx._check(self.ctx.lib.smelt_cuda_enqueue_prefill_rows(self.ctx.h, self.prefill_records, len(self.prefill_records), tokens.ctypes.data_as(C.c_void_p), len(tokens),
+                                                                     int(start_pos), rows.ctypes.data_as(C.c_void_p), len(rows)))
+
+    def prefill_by_table(self, tokens, start_pos: int = 0) -> int:
+        """Prompt tokens a chunk at a time; only the last chunk runs the head.  Returns the argmax after the last token."""
+        tokens = np.ascontiguousarray(np.asarray(tokens).reshape(-1), dtype=np.int32)
+        for t0 in range(0, len(tokens), self.prefill_chunk):
+            part = np.ascontiguousarray(tokens[t0:t0 + self.prefill_chunk])
+            self._enqueue_chunk(part, start_pos + t0, [len(part) - 1] if t0 + len(part) == len(tokens) else [])
+        out = np.zeros(1, np.int32)
+        self.ctx._check(self.ctx.lib.smelt_cuda_read_slot(self.ctx.h, ARGMAX_SLOT, 0, out.ctypes.data_as(C.c_void_p), 4))
+        return int(out[0])
+
+    def prefill(self, tokens, start_pos: int = 0, chunk: int = 0) -> int:
+        return self.prefill_by_table(tokens, start_pos)
+
+    def feed(self, tokens, start_pos: int, want=()) -> np.ndarray:
+        """The sequence's next tokens, at positions ``start_pos ...``: one through the decode graph,
+        several through the prompt-chunk table.  Logits ``[len(want), vocab]`` of the places asked for."""
+        tokens = np.ascontiguousarray(np.asarray(tokens).reshape(-1), dtype=np.int32)
+        want = [int(w) for w in want]
+        if any(not 0 <= w < len(tokens) for w in want):
+            raise ValueError("a wanted place is outside the tokens")
+        if len(tokens) == 1:
+            if not self.graph_ready:
+                self.build_graph()
+            self.graph_step(int(tokens[0]), start_pos)
+            return np.repeat(self.logits(1), len(want), 0)
+        out = np.empty((len(want), self.desc.vocab), np.float32)
+        for t0 in range(0, len(tokens), self.prefill_chunk):
+            part = np.ascontiguousarray(tokens[t0:t0 + self.prefill_chunk])
+            inside = [i for i, w in enumerate(want) if t0 <= w < t0 + len(part)]
+            rows = sorted({want[i] - t0 for i in inside})
+            self._enqueue_chunk(part, start_pos + t0, rows)
+            if rows:
+                got = self.logits(len(rows))
+                for i in inside:
+                    out[i] = got[rows.index(want[i] - t0)]
+        return out
+
+    def graph_step(self, token: int, position: int) -> int:
+        tok, out = np.array([token], np.int32), np.zeros(1, np.int32)
+        self.ctx._check(self.ctx.lib.smelt_cuda_graph_step(self.ctx.h, tok.ctypes.data_as(C.c_void_p), int(position), out.ctypes.data_as(C.c_void_p)))
+        return int(out[0])
+
+    def generate(self, prompt, n_decode: int, use_graph: bool = True) -> np.ndarray:
+        """The prompt through the prompt-chunk table, then greedy steps; ids ``[n_decode, 1]``."""
+        prompt = np.asarray(prompt, dtype=np.int32).reshape(-1)
+        out = np.zeros((n_decode, 1), np.int32)
+        if n_decode == 0:
+            return out
+        if use_graph and not self.graph_ready:
+            self.build_graph()
+        out[0] = self.prefill_by_table(prompt)
+        if use_graph and n_decode > 1:
+            self.graph_seed(out[0], len(prompt))
+            out[1:] = self.graph_decode(n_decode - 1, read=True)
+            return out
+        for i in range(1, n_decode):
+            out[i] = self.decode_step(out[i - 1], len(prompt) + i - 1)
+        return out
+
+    def cache_slots(self) -> list[int]:
+        first, n = C.c_int32(0), C.c_int32(0)
+        self.ctx._check(self.ctx.lib.smelt_cuda_dense_cache_slots(C.byref(self.desc), C.byref(first), C.byref(n)))
+        return list(range(first.value, first.value + n.value))
+
+    def reset_cache(self):
+        """Not needed between sequences: a row is written before a position that sees it is reached."""
+        for s in self.cache_slots():
+            self.ctx.call("zero_slot", s)
+
+    def kv_slots(self):
+        return (capi.KvSlot * 0)()
+
+    def state_slots(self):
+        return self.cache_slots()  # rings and block means: copied whole, restored only at their full length
 
 
 class Snapshot:
