@@ -346,6 +346,42 @@ SMELT_CUDA_API smelt_status smelt_cuda_build_dense_prefill_table(smelt_cuda_ctx*
  * snapshots they are position-less state (a ring cannot be cut to a shorter length). */
 SMELT_CUDA_API smelt_status smelt_cuda_dense_cache_slots(const smelt_dense_desc* desc, int32_t* first_slot, int32_t* n_slots);
 
+/* Typed launchers of those tables' kernels.  precision: SMELT_DENSE_BF16 or SMELT_DENSE_F32, the type T of a chunk's
+ * activations and of the caches.  Weights are bf16, cols a multiple of 64 with zero padding.
+ * mode: 0 y0 = fp32 product, 1 y0 += product (fp32), 2 rows below split to y0, the others through xIELU to y1, both in T
+ * (dense_matvec: fp32, and modes 0 and 1 only; rows from split on always go through xIELU to y1). */
+SMELT_CUDA_API smelt_status smelt_cuda_dense_gemm(smelt_cuda_ctx* ctx, int precision, int mode, const void* w_dev, const void* x_dev, void* y0_dev,
+                                                  void* y1_dev, int rows, int cols, int m, int split, int ld0, int ld1, float rising, float falling);
+/* One fp32 activation row; x is [xa (ka values); xb] when xb is given; norm_width > 0 scales the product by gain / rms(x). */
+SMELT_CUDA_API smelt_status smelt_cuda_dense_matvec(smelt_cuda_ctx* ctx, int mode, const void* w_dev, const void* xa_dev, const void* xb_dev, int ka,
+                                                    void* y0_dev, void* y1_dev, int rows, int cols, int split, int norm_width, float gain, float eps,
+                                                    float rising, float falling);
+SMELT_CUDA_API smelt_status smelt_cuda_embed_positions(smelt_cuda_ctx* ctx, const void* table_dev, const void* tokens_dev, const void* positions_dev,
+                                                       void* x_dev, void* x0_dev, int width, int ld, int m, uint32_t vocab, uint32_t max_positions,
+                                                       float scale, uint32_t position);
+SMELT_CUDA_API smelt_status smelt_cuda_scalar_norm_rows(smelt_cuda_ctx* ctx, int precision, const void* x_dev, const void* rows_dev, void* out_dev,
+                                                        int width, int ld, int m, float gain, float eps);
+SMELT_CUDA_API smelt_status smelt_cuda_pair_rows(smelt_cuda_ctx* ctx, int precision, const void* x_dev, const void* x0_dev, void* out_dev, int ld, int m);
+/* Attention over a window and pooled blocks.  A K (V) cache is [kv_heads, ring + blocks, row] of T, row = dim (vdim) padded
+ * with zeros to 64, 128, 256 or a multiple of 64 beyond; position p lives in row p % ring, block b in row ring + b; ring must
+ * be at least max(window, pool) + m - 1.  u: [m, heads dim + kv_heads (dim + vdim)] projections q | k | v, q: [m, heads, row]
+ * normed queries, z: [m, ldz], all in T (window_decode: fp32, q is scratch). */
+typedef struct {
+    int32_t heads, kv_heads, dim, vdim;
+    uint32_t window, pool, ring, blocks;
+    float scale, softcap, eps;
+} smelt_window_desc;
+SMELT_CUDA_API smelt_status smelt_cuda_window_append(smelt_cuda_ctx* ctx, int precision, const smelt_window_desc* desc, const void* u_dev,
+                                                     const void* q_norm_dev, const void* k_norm_dev, void* k_cache_dev, void* v_cache_dev, void* q_dev,
+                                                     int m, uint32_t position);
+SMELT_CUDA_API smelt_status smelt_cuda_window_pool(smelt_cuda_ctx* ctx, int precision, const smelt_window_desc* desc, void* k_cache_dev,
+                                                   void* v_cache_dev, int m, uint32_t position);
+SMELT_CUDA_API smelt_status smelt_cuda_window_attention(smelt_cuda_ctx* ctx, int precision, const smelt_window_desc* desc, const void* q_dev,
+                                                        void* k_cache_dev, void* v_cache_dev, void* z_dev, int ldz, int m, uint32_t position);
+SMELT_CUDA_API smelt_status smelt_cuda_window_decode(smelt_cuda_ctx* ctx, int precision, const smelt_window_desc* desc, const void* u_dev,
+                                                     const void* q_norm_dev, const void* k_norm_dev, void* k_cache_dev, void* v_cache_dev, void* q_dev,
+                                                     void* z_dev, uint32_t position);
+
 /* The pipeline names of the table smelt_cuda_build_prefill_table writes, in the order of the indices a table built
  * without a context carries (0, 1, ...): newline separated, as smelt_cuda_decoder_pipelines reports the decode table's. */
 SMELT_CUDA_API smelt_status smelt_cuda_prefill_pipelines(const smelt_decoder_desc* desc, char* out, size_t out_bytes, size_t* needed_bytes);

@@ -108,6 +108,12 @@ class DenseDesc(C.Structure):
                 ("final_gain", C.c_float), ("embedding", C.c_uint64), ("positions", C.c_uint64), ("loop_in", C.c_uint64), ("lm_head", C.c_uint64)]
 
 
+class WindowDesc(C.Structure):
+    """``smelt_window_desc``: attention over a sliding window and pooled blocks."""
+    _fields_ = [("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("window", C.c_uint32), ("pool", C.c_uint32),
+                ("ring", C.c_uint32), ("blocks", C.c_uint32), ("scale", C.c_float), ("softcap", C.c_float), ("eps", C.c_float)]
+
+
 class PackageOptions(C.Structure):
     _fields_ = [("context_capacity", C.c_uint32), ("context_limit", C.c_uint32)]
 

@@ -1,6 +1,7 @@
 // Device side of the flash-decode attention kernel (see attention.cu for the description).
 #pragma once
 #include <cooperative_groups.h>
+#include <cuda_bf16.h>
 
 #include "glue.h"
 #include "rope.cuh"
@@ -22,6 +23,22 @@ __device__ __forceinline__ uint32_t movmatrix_trans(uint32_t a) {
     asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(d) : "r"(a));
     return d;
 }
+
+// The 16-bit element a tile works on: its MMA and its packing.
+template <class E> struct TileElem;
+template <> struct TileElem<__half> {
+    static __device__ __forceinline__ void mma(float c[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) { mma16816(c, a0, a1, a2, a3, b0, b1); }
+    static __device__ __forceinline__ uint32_t pack(float x, float y) { return h2_as_u32(__floats2half2_rn(x, y)); }
+    static __device__ __forceinline__ float2 unpack(uint32_t v) { return __half22float2(u32_as_h2(v)); }
+};
+template <> struct TileElem<__nv_bfloat16> {
+    static __device__ __forceinline__ void mma(float c[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) { mma16816_bf16(c, a0, a1, a2, a3, b0, b1); }
+    static __device__ __forceinline__ uint32_t pack(float x, float y) {
+        const __nv_bfloat162 v = __floats2bfloat162_rn(x, y);
+        return *reinterpret_cast<const uint32_t*>(&v);
+    }
+    static __device__ __forceinline__ float2 unpack(uint32_t v) { return make_float2(__uint_as_float(v << 16), __uint_as_float(v & 0xFFFF0000u)); }
+};
 
 // out = sum_s exp2(m_s - M) O_s / sum_s exp2(m_s - M) l_s over the splits of `heads` consecutive
 // query heads starting at qh0, splits in index order.  The (max, sum) pairs are staged in shared
@@ -73,19 +90,11 @@ __device__ __forceinline__ void key_range(const AttnDev& p, uint32_t& seq_start,
     if (p.a.sliding_window > 0 && p.a.sliding_window < seq_len) seq_start = seq_len - p.a.sliding_window;
 }
 
-// One (split, KV head, sequence) work item by one CTA of kAttnThreads threads.  Sync is called
-// once by every thread before the first read of q or the caches (see affine_imma.cuh).
-// One 16-key tile, first half: S^T = K . Q^T from the K unit's pieces (ku: piece p of lane l at
-// p * 512 + l * 16, already offset to this lane), then the online softmax of the tile's columns.
-// valid_a / valid_b: this thread's keys g and g + 8 of the tile take part.  Leaves P^T as fp16
-// high and low parts in B-operand layout (pb0, pb1, pl0, pl1) and rescales m_run, l_run, o.
-template <int D, int NH>
-__device__ __forceinline__ void tile_scores_softmax(const unsigned char* ku, const uint32_t (&qf)[NH][D / 8], bool valid_a, bool valid_b,
-                                                    float scale2, float (&m_run)[NH][2], float (&l_run)[NH][2], float (&o)[NH][D / 16][4],
-                                                    uint32_t (&pb0)[NH], uint32_t (&pb1)[NH], uint32_t (&pl0)[NH], uint32_t (&pl1)[NH]) {
-    constexpr int MT = D / 16, KJ = D / 32;
-    // ── S^T = K · Q^T ──
-    float s[NH][4];
+// One 16-key tile: S^T = K . Q^T from the K unit's pieces (ku: piece p of lane l at p * 512 + l * 16,
+// already offset to this lane).  Thread (g, t) gets keys g and g + 8 of heads 2t and 2t + 1.
+template <int D, int NH, class E = __half>
+__device__ __forceinline__ void tile_scores(const unsigned char* ku, const uint32_t (&qf)[NH][D / 8], float (&s)[NH][4]) {
+    constexpr int KJ = D / 32;
 #pragma unroll
     for (int nh = 0; nh < NH; ++nh) s[nh][0] = s[nh][1] = s[nh][2] = s[nh][3] = 0.f;
 #pragma unroll
@@ -93,10 +102,22 @@ __device__ __forceinline__ void tile_scores_softmax(const unsigned char* ku, con
         const uint4 ka = *reinterpret_cast<const uint4*>(ku + (2 * j) * 512), kb = *reinterpret_cast<const uint4*>(ku + (2 * j + 1) * 512);
 #pragma unroll
         for (int nh = 0; nh < NH; ++nh) {
-            mma16816(s[nh], ka.x, kb.x, ka.y, kb.y, qf[nh][4 * j + 0], qf[nh][4 * j + 1]);
-            mma16816(s[nh], ka.z, kb.z, ka.w, kb.w, qf[nh][4 * j + 2], qf[nh][4 * j + 3]);
+            TileElem<E>::mma(s[nh], ka.x, kb.x, ka.y, kb.y, qf[nh][4 * j + 0], qf[nh][4 * j + 1]);
+            TileElem<E>::mma(s[nh], ka.z, kb.z, ka.w, kb.w, qf[nh][4 * j + 2], qf[nh][4 * j + 3]);
         }
     }
+}
+
+// Its first half with the online softmax of the tile's columns.
+// valid_a / valid_b: this thread's keys g and g + 8 of the tile take part.  Leaves P^T as fp16
+// high and low parts in B-operand layout (pb0, pb1, pl0, pl1) and rescales m_run, l_run, o.
+template <int D, int NH>
+__device__ __forceinline__ void tile_scores_softmax(const unsigned char* ku, const uint32_t (&qf)[NH][D / 8], bool valid_a, bool valid_b,
+                                                    float scale2, float (&m_run)[NH][2], float (&l_run)[NH][2], float (&o)[NH][D / 16][4],
+                                                    uint32_t (&pb0)[NH], uint32_t (&pb1)[NH], uint32_t (&pl0)[NH], uint32_t (&pl1)[NH]) {
+    constexpr int MT = D / 16;
+    float s[NH][4];
+    tile_scores<D, NH>(ku, qf, s);
 
     // ── online softmax per query head (columns 2t, 2t+1 of the tile) ──
 #pragma unroll
@@ -134,7 +155,7 @@ __device__ __forceinline__ void tile_scores_softmax(const unsigned char* ku, con
 }
 
 // Second half: O^T += V^T . P^T from the V unit's pieces (vu, same addressing).
-template <int D, int NH>
+template <int D, int NH, class E = __half>
 __device__ __forceinline__ void tile_weighted_sum(const unsigned char* vu, float (&o)[NH][D / 16][4], const uint32_t (&pb0)[NH],
                                                   const uint32_t (&pb1)[NH], const uint32_t (&pl0)[NH], const uint32_t (&pl1)[NH]) {
     constexpr int VC = D / 64;
@@ -152,8 +173,8 @@ __device__ __forceinline__ void tile_weighted_sum(const unsigned char* vu, float
             const uint32_t a2 = __byte_perm(r2[e], r3[e], 0x5410), a3 = __byte_perm(r2[e], r3[e], 0x7632);
 #pragma unroll
             for (int nh = 0; nh < NH; ++nh) {
-                mma16816(o[nh][4 * c + e], a0, a1, a2, a3, pb0[nh], pb1[nh]);
-                mma16816(o[nh][4 * c + e], a0, a1, a2, a3, pl0[nh], pl1[nh]);
+                TileElem<E>::mma(o[nh][4 * c + e], a0, a1, a2, a3, pb0[nh], pb1[nh]);
+                TileElem<E>::mma(o[nh][4 * c + e], a0, a1, a2, a3, pl0[nh], pl1[nh]);
             }
         }
     }
@@ -182,6 +203,8 @@ __host__ __device__ constexpr size_t attn_smem_bytes() {
 }
 
 
+// One (split, KV head, sequence) work item by one CTA of kAttnThreads threads.  Sync is called
+// once by every thread before the first read of q or the caches (see affine_imma.cuh).
 template <int D, int NH, int NU, class Sync>
 __device__ __forceinline__ void attn_decode_body(const AttnDev& p, float* smem_f, int split, int kvh, int b, Sync sync) {
     constexpr int MT = D / 16;  // m-tiles of O^T

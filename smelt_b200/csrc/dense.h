@@ -102,9 +102,6 @@ struct WindowArgs {
     void* z;                    // [m, ldz]: the heads' outputs in columns [0, heads vdim)
     int ldz;
     int sm_count;
-    void* scratch;
-    size_t scratch_bytes;
-    int* counters;
     DevDyn dyn;
 };
 inline int window_padded(int d) { return d <= 64 ? 64 : d <= 128 ? 128 : d <= 256 ? 256 : (d + 63) / 64 * 64; }

@@ -796,7 +796,7 @@ smelt_status run_dense(Interp& in, const Pipeline& p, const Resolved& r) {
     const size_t us = p.kind == PK_WINDOW_DECODE ? 4 : es;
     NEED_BYTES(3, rows * a.kp * es); NEED_BYTES(4, rows * a.vp * es);
     a.k_cache = r.buf[3].ptr; a.v_cache = r.buf[4].ptr;
-    a.sm_count = ctx->sm_count; a.scratch = ctx->attn_scratch; a.scratch_bytes = ctx->attn_scratch_bytes; a.counters = ctx->attn_counters;
+    a.sm_count = ctx->sm_count;
     if (p.kind == PK_WINDOW_POOL) return check_cuda(ctx, launch_window_pool(l, type, a), p.name.c_str());
     NEED_BUF(5); NEED_BYTES(5, (size_t)a.m * a.heads * a.kp * us);
     a.q = r.buf[5].ptr;

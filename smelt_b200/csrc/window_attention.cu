@@ -4,17 +4,17 @@
 // Score s = (q . k) scale, then softcap tanh(s / softcap); the softmax has one more in its
 // denominator (a sink with score 0 and no value).  Tokens of the window and pooled blocks share
 // one softmax.  Norms, scores, weights and sums are fp32.
+//
+// The kernels here take any head size, softcap (or none) and cache type; with a bf16 cache, heads
+// of up to 256 and a softcap the tensor-core kernels of window_decode.cu and window_prefill.cu run
+// instead.
 #include <algorithm>
 
-#include "dense.h"
+#include "window.cuh"
 
 namespace smelt {
 
 namespace {
-
-// The blocks a query at position i sees: [0, n).
-__device__ __forceinline__ uint32_t visible_blocks(uint32_t i, uint32_t window, uint32_t pool) { return i + 1u >= window ? (i + 1u - window) / pool : 0u; }
-__device__ __forceinline__ uint32_t window_start(uint32_t i, uint32_t window) { return i + 1u > window ? i + 1u - window : 0u; }
 
 // One warp per head of a token: query heads normed to q, key heads normed into the ring, value
 // heads copied into it.
@@ -51,18 +51,6 @@ __global__ void __launch_bounds__(256) window_append_kernel(const WindowArgs a) 
         TC* dst = static_cast<TC*>(a.k_cache) + ((item - H) * head_rows + slot) * a.kp;
         for (int d = lane; d < a.dim; d += 32) dst[d] = from_f32<TC>(to_f32(src[d]) * f * to_f32(w[d]));
     }
-}
-
-// Mean of a block's rows as the cache holds them, in position order.
-template <class TC>
-__device__ __forceinline__ float block_mean(const TC* head, uint32_t first, uint32_t pool, uint32_t ring, int pitch, int d) {
-    float sum = 0.f;
-    uint32_t slot = first % ring;
-    for (uint32_t j = 0; j < pool; ++j) {
-        sum += to_f32(head[(size_t)slot * pitch + d]);
-        slot = slot + 1u == ring ? 0u : slot + 1u;
-    }
-    return sum / (float)pool;
 }
 
 template <class TC>
@@ -179,12 +167,18 @@ cudaError_t launch_window_attention(const Launch& l, DenseType type, WindowArgs 
     if (bad_geometry(a)) return cudaErrorInvalidValue;
     a.dyn = dev_dyn(l);
     if (type == kDenseF32) return simple_t<float, float>(l, a);
+    if (!a.u_f32 && window_tiled(a)) return launch_window_prefill_tiled(l, a);
     return a.u_f32 ? simple_t<bf16, float>(l, a) : simple_t<bf16, bf16>(l, a);
 }
 
 cudaError_t launch_window_decode(const Launch& l, DenseType type, WindowArgs a, int* launches) {
     if (a.m != 1) return cudaErrorInvalidValue;
     a.u_f32 = 1;
+    if (type == kDenseBf16 && !bad_geometry(a) && window_tiled(a)) {
+        a.dyn = dev_dyn(l);
+        *launches = 1;
+        return launch_window_decode_tiled(l, a);
+    }
     *launches = 3;
     cudaError_t e = launch_window_append(l, type, a);
     if (e == cudaSuccess) e = launch_window_pool(l, type, a);
