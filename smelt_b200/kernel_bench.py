@@ -251,6 +251,67 @@ class Bench:
         for t in states + [dq, b, a, a_log, dt, out]:
             t.free()
 
+    # ── dense 16-bit weights ──
+    def bf16_weights(self, tag, rows, cols):
+        """Random signs and mantissas at one small magnitude, as bf16 bit patterns (quick to make at any size)."""
+        bits = synth.rng_for(6, tag).integers(0, 1 << 16, (rows, cols), dtype=np.uint16)
+        return (bits & np.uint16(0x807F)) | np.uint16((127 - 6) << 7)
+
+    def dense_matvec(self, config, rows, cols, split=None, add=False):
+        """A decode step's projection: norm factor and xIELU past `split`, or added to the residual."""
+        ctx = self.ctx
+        alg = rows * cols * 2 + cols * 4 + rows * 4 * (2 if add else 1)
+        n = copies_for(alg)
+        w = [ctx.to_device(self.bf16_weights(f"dm{rows}", rows, cols)) for _ in range(n)]
+        x, y, y1 = ctx.to_device(np.ones(cols, np.float32)), ctx.alloc(rows * 4).fill(0), ctx.alloc(rows * 4).fill(0)
+        split = rows if split is None else split
+        def enqueue():
+            for wi in w:
+                ctx.call("dense_matvec", int(add), wi, x, None, 0, y, y1, rows, cols, split, 0 if add else cols, 1.0, 1e-6, 0.7, 1.2)
+        self.run(config, "dense_matvec" + (" + residual" if add else " (norm, xIELU)" if split < rows else " (norm)"), f"{rows}x{cols}", 1, alg, n, enqueue)
+        for b in (*w, x, y, y1):
+            b.free()
+
+    def dense_gemm(self, config, rows, cols, m, split=None, add=False):
+        ctx = self.ctx
+        alg = rows * cols * 2 + m * cols * 2 + m * rows * (8 if add else 2)
+        n = copies_for(alg, cap=16)
+        w = [ctx.to_device(self.bf16_weights(f"dg{rows}", rows, cols)) for _ in range(n)]
+        x, y, y1 = ctx.to_device(self.bf16_weights("dgx", m, cols)), ctx.alloc(m * rows * 4).fill(0), ctx.alloc(m * rows * 2).fill(0)
+        split = rows if split is None else split
+        def enqueue():
+            for wi in w:
+                ctx.call("dense_gemm", 0, 1 if add else 2, wi, x, y, y1, rows, cols, m, split, rows, rows, 0.7, 1.2)
+        self.run(config, "dense_gemm" + (" + residual" if add else " (xIELU)"), f"{rows}x{cols}", m, alg, n, enqueue, flops=2.0 * rows * cols * m)
+        for b in (*w, x, y, y1):
+            b.free()
+
+    def window(self, config, n_q, n_kv, d, window, pool, position, m=1):
+        """Window + pooled-block attention at `position`: a decode step (m 1) or a prompt chunk that ends there."""
+        ctx = self.ctx
+        blocks, start = (position + 1) // pool, position + 1 - m
+        ring = -(-(max(window, pool) + m) // 64) * 64
+        desc = capi.WindowDesc(n_q, n_kv, d, d, window, pool, ring, blocks, 1 / np.sqrt(d), 20.0, 1e-6)
+        seen = [min(i + 1, window) + max(0, (i + 1 - window) // pool) for i in range(start, position + 1)]
+        keys = seen[-1] + (m - 1 if m > 1 else 0)  # rows of the cache the launch reads
+        alg = 2 * n_kv * d * 2 * keys + (2 * m * n_q * d * 2 if m > 1 else (2 * n_q + 2 * n_kv) * d * 4)
+        n = copies_for(alg, cap=48)
+        caches = [[ctx.to_device(self.bf16_weights(f"wc{t}", n_kv * (ring + blocks), d)) for t in "kv"] for _ in range(n)]
+        norm, es = ctx.to_device(np.full(d, 0x3F80, np.uint16)), 2 if m > 1 else 4
+        q = ctx.to_device(self.bf16_weights("wq", m * n_q, d) if m > 1 else np.zeros(n_q * d, np.float32))
+        u, z = ctx.to_device(np.ones((n_q + 2 * n_kv) * d, np.float32)), ctx.alloc(m * n_q * d * es)
+        def enqueue():
+            for k, v in caches:
+                if m == 1:
+                    ctx.call("window_decode", 0, C.byref(desc), u, norm, norm, k, v, q, z, position)
+                else:
+                    ctx.call("window_attention", 0, C.byref(desc), q, k, v, z, n_q * d, m, start)
+        self.run(config, "window_decode (norms, append, attention)" if m == 1 else "window_attention (prompt chunk)",
+                 f"{n_q}q x {n_kv}kv x d{d}, window {window}, pool {pool}, " + (f"position {position}" if m == 1 else f"{m} positions from {start}"), 1, alg, n, enqueue,
+                 flops=4.0 * n_q * d * sum(seen))
+        for b in (*[c for kv in caches for c in kv], norm, q, u, z):
+            b.free()
+
     def lm_head(self, config, vocab, hidden):
         ctx = self.ctx
         w = ctx.to_device(synth.normal_f16(4, "head", (vocab, hidden), 0.02))

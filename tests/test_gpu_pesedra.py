@@ -50,8 +50,15 @@ def seen_as(a, precision):
 
 
 def worst(got, want):
+    """Largest difference over the reference's root mean square."""
     want = np.asarray(want, np.float64)
     return float(np.max(np.abs(got - want)) / np.sqrt(np.mean(want * want)))
+
+
+def worst_row(got, want):
+    """The same for the root-mean-square difference of a row (the last axis): the measure for 16-bit outputs."""
+    want = np.asarray(want, np.float64)
+    return float(np.max(np.sqrt(np.mean((got - want) ** 2, -1))) / np.sqrt(np.mean(want * want)))
 
 
 # ── projections ─────────────────────────────────────────────────────────────
@@ -66,7 +73,7 @@ def test_dense_gemm(ctx, rows, cols, m, precision):
     w, x = cases.round_bf16(g.standard_normal((rows, cols)) / np.sqrt(cols)), seen_as(g.standard_normal((m, cols)), precision)
     want = x @ w.T.astype(np.float64)
     dw, dx = put(ctx, w), put(ctx, x, precision)
-    tol = 3e-5
+    tol = 1e-4
     ld = rows + 3
     y = put(ctx, np.full((m, ld), 7.0), "float32")
     ctx.call("dense_gemm", code, 0, dw, dx, y, None, rows, cols, m, rows, ld, 0, 0.0, 0.0)
@@ -81,7 +88,7 @@ def test_dense_gemm(ctx, rows, cols, m, precision):
     rest = want[:, split:]
     neg = np.minimum(rest, 0)
     act = np.where(rest > 0, rising * rest * rest, falling * (np.expm1(neg) - neg)) + rest / 2
-    out_tol = 3e-5 if precision == "float32" else 1.0 / 256
+    out_tol = 1e-4 if precision == "float32" else 1.0 / 256
     lhs, rhs = take(y0, (m, split + 1), precision), take(y1, (m, rows), precision)
     assert np.all(np.abs(lhs[:, :split] - want[:, :split]) <= out_tol * (np.abs(want[:, :split]) + 0.05))
     assert np.all(np.abs(rhs[:, :rows - split] - act) <= out_tol * (np.abs(act) + 0.05)) and (rhs[:, rows - split:] == 5.0).all()
@@ -186,9 +193,11 @@ class Window:
         n, H, G, d, dv = len(u), self.H, self.G, self.dim, self.vdim
         return u[:, :H * d].reshape(n, H, d), u[:, H * d:(H + G) * d].reshape(n, G, d), u[:, (H + G) * d:].reshape(n, G, dv)
 
-    def want(self, u):
-        """The restatement on the values as the device stores them."""
-        q, k, v = self.split(seen_as(u, self.precision))
+    def want(self, u, cuts=None):
+        """The restatement on the values as the device stores them: a decoded token's projections stay fp32."""
+        chunked = np.repeat([c > 1 for c in cuts or [len(u)]], cuts or [len(u)])[:, None]
+        q, k, v = self.split(np.where(chunked, seen_as(u, self.precision), seen_as(u, "float32")))
+        v = seen_as(v, self.precision)
         q, k = (seen_as(ref.head_rms_norm(x, w, self.desc.eps), self.precision) for x, w in ((q, self.qn), (k, self.kn)))
         d = self.desc
         if d.softcap <= 0:  # the restatement always caps; a huge cap is none
@@ -210,12 +219,13 @@ def test_window_attention(ctx, geometry, precision, cut):
     n = sum(CUTS[cut])
     w = Window(ctx, precision, H, G, dim, vdim, window, pool, dim ** -0.5 * 2.0, 12.0, positions=n + 3, chunk=64, seed=cut)
     u = np.random.default_rng(cut + dim).standard_normal((n, H * dim + G * (dim + vdim)))
-    want = w.want(u)
+    want = w.want(u, CUTS[cut])
     got, at = [], 0
     for c in CUTS[cut]:
         got.append(w.feed(u[at:at + c]))
         at += c
-    assert worst(np.concatenate(got), want) < (2e-5 if precision == "float32" else 0.03)
+    got = np.concatenate(got)
+    assert worst(got, want) < 2e-5 if precision == "float32" else worst_row(got, want) < 0.015
 
 
 @pytest.mark.parametrize("precision", PRECISIONS)
@@ -225,7 +235,8 @@ def test_softcaps(ctx, precision, softcap):
     w = Window(ctx, precision, 4, 2, 64, 64, 30, 4, 0.6, softcap, positions=130, chunk=64, seed=9)
     u = np.random.default_rng(5).standard_normal((96, 4 * 64 + 2 * 128))
     got = np.concatenate([w.feed(u[:64]), *[w.feed(u[i:i + 1]) for i in range(64, 96)]])
-    assert worst(got, w.want(u)) < (1e-4 if precision == "float32" else 0.06)
+    want = w.want(u, [64] + [1] * 32)
+    assert worst(got, want) < 1e-4 if precision == "float32" else worst_row(got, want) < 0.03
 
 
 def standout(w, n, query, keys, value):
@@ -300,7 +311,7 @@ def open_decoder(ctx, name, precision, max_chunk=64, seed=0, **kw):
     return arch.decoder(ctx, arch.parse(cfg), checkpoint.TensorFile(cases.stored(t)), precision=precision, max_chunk=max_chunk, **kw), ref.Pesedra(cfg, t)
 
 
-LIMIT = {"float32": 1e-4, "bfloat16": 0.12}
+LIMIT = {"float32": 1e-5, "bfloat16": 0.025}  # of worst_row
 _reference = {}
 
 
@@ -329,7 +340,7 @@ def test_model_whole_portions_and_decoded(ctx, name, precision):
     toks = cases.tokens(cases.ALL[name], n)
     want = reference_logits(name, m, toks)
     for cuts in ([n], [2] * 10 + [n - 20], [3, 17, 1, 1, 50, 2, 33, 1, 1, 1, n - 110], [n - 80] + [1] * 80, [1] * n):
-        err = worst(run_cuts(dec, toks, cuts), want)
+        err = worst_row(run_cuts(dec, toks, cuts), want)
         assert err < LIMIT[precision], (cuts[:6], err)
 
 
@@ -339,7 +350,7 @@ def test_cache_is_used_again_without_clearing(ctx, precision):
     dec, m = open_decoder(ctx, "mixed", precision)
     for n, seed, cuts in ((140, 3, [139, 1]), (1, 4, [1]), (23, 5, [2, 21]), (90, 6, [60] + [1] * 30), (140, 3, [1] * 20 + [120])):
         toks = cases.tokens(cases.MIXED, n, seed)
-        assert worst(run_cuts(dec, toks, cuts), reference_logits("mixed", m, toks)) < LIMIT[precision]
+        assert worst_row(run_cuts(dec, toks, cuts), reference_logits("mixed", m, toks)) < LIMIT[precision]
 
 
 def test_only_wanted_rows(ctx):
@@ -429,5 +440,5 @@ def test_trace_run_program(ctx, tmp_path, precision):
     lb = m.feed(b)
     read = lambda i: np.fromfile(out / f"{i}.f32", "<f4").reshape(-1, cfg["vocab"])
     for i, want in ((0, la[[0, 76]]), (1, la[[97]]), (3, la[[99]]), (4, lb[[29]])):
-        assert worst(read(i), want) < LIMIT[precision]
+        assert worst_row(read(i), want) < LIMIT[precision]
     assert not (out / "2.f32").exists()
