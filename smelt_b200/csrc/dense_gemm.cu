@@ -26,12 +26,9 @@ namespace smelt {
 
 namespace {
 
-template <int MODE, class T>
-__device__ __forceinline__ void dense_store(const DenseOut& o, int token, int row, float v) {
-    if (MODE == kDenseStoreF32) static_cast<float*>(o.y0)[(size_t)token * o.ld0 + row] = v;
-    else if (MODE == kDenseAddF32) static_cast<float*>(o.y0)[(size_t)token * o.ld0 + row] += v;
-    else if (row < o.split) static_cast<T*>(o.y0)[(size_t)token * o.ld0 + row] = from_f32<T>(v);
-    else static_cast<T*>(o.y1)[(size_t)token * o.ld1 + (row - o.split)] = from_f32<T>(xielu(v, o.rising, o.falling));
+// xIELU for a bf16 result: the exponential's error (a few 2^-24 absolute near zero) is far below the result's rounding.
+__device__ __forceinline__ float xielu_bf16(float z, float rising, float falling) {
+    return fmaf(0.5f, z, z > 0.f ? rising * z * z : falling * (__expf(z) - 1.f - z));
 }
 
 // ── tcgen05 ─────────────────────────────────────────────────────────────────
@@ -75,6 +72,7 @@ __global__ void __launch_bounds__(kGemmThreads, 1) gemm_bf16_kernel(const __grid
                                                                     const GemmPlan plan) {
     constexpr int kStages = gemm_stages(BN);
     constexpr uint32_t kStageBytes = gemm_stage_bytes(BN), kTmemCols = 2 * BN < 32 ? 32 : 2 * BN;
+    constexpr int kChunk = BN < 32 ? BN : 32;
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
     __shared__ uint64_t full[kStages], empty[kStages], acc_full[2], acc_empty[2];
@@ -187,12 +185,13 @@ __global__ void __launch_bounds__(kGemmThreads, 1) gemm_bf16_kernel(const __grid
             bool finish = true;
             if (plan.ksplit > 1) {
                 float* mine = a.part_scratch + (size_t)u * (BN * kBlockRows);
-                for (int c0 = 0; c0 < cnt; c0 += 8) {
-                    uint32_t v[8];
-                    tmem_ld8(lane_base + buf * BN + c0, v);
+                for (int c0 = 0; c0 < cnt; c0 += kChunk) {
+                    uint32_t v[kChunk / 8][8];
+#pragma unroll
+                    for (int j = 0; j < kChunk / 8; ++j) tmem_ld8(lane_base + buf * BN + c0 + 8 * j, v[j]);
                     tmem_wait_ld();
 #pragma unroll
-                    for (int j = 0; j < 8; ++j) __stcg(mine + (size_t)(c0 + j) * kBlockRows + r, __uint_as_float(v[j]));
+                    for (int j = 0; j < kChunk; ++j) __stcg(mine + (size_t)(c0 + j) * kBlockRows + r, __uint_as_float(v[j / 8][j % 8]));
                 }
                 __threadfence();
                 asm volatile("bar.sync 1, %0;" ::"n"(kEpilogueThreads) : "memory");
@@ -206,36 +205,50 @@ __global__ void __launch_bounds__(kGemmThreads, 1) gemm_bf16_kernel(const __grid
             }
             if (finish) {
                 const float* parts = a.part_scratch + (size_t)tile * plan.ksplit * (BN * kBlockRows) + r;
-                for (int c0 = 0; c0 < cnt; c0 += 8) {
-                    float v[8];
+                for (int c0 = 0; c0 < cnt; c0 += kChunk) {  // positions, kChunk at a time: their loads are in flight together
+                    float v[kChunk];
                     if (plan.ksplit > 1) {
 #pragma unroll
-                        for (int j = 0; j < 8; ++j) v[j] = 0.f;
-                        for (int z = 0; z < plan.ksplit; ++z)
+                        for (int j = 0; j < kChunk; ++j) v[j] = __ldcg(parts + (size_t)(c0 + j) * kBlockRows);
+                        for (int z = 1; z < plan.ksplit; ++z)
 #pragma unroll
-                            for (int j = 0; j < 8; ++j) v[j] += __ldcg(parts + (size_t)z * (BN * kBlockRows) + (size_t)(c0 + j) * kBlockRows);
+                            for (int j = 0; j < kChunk; ++j) v[j] += __ldcg(parts + (size_t)z * (BN * kBlockRows) + (size_t)(c0 + j) * kBlockRows);
                     } else {
-                        uint32_t w[8];
-                        tmem_ld8(lane_base + buf * BN + c0, w);
+                        uint32_t w[kChunk / 8][8];
+#pragma unroll
+                        for (int j = 0; j < kChunk / 8; ++j) tmem_ld8(lane_base + buf * BN + c0 + 8 * j, w[j]);
                         tmem_wait_ld();
 #pragma unroll
-                        for (int j = 0; j < 8; ++j) v[j] = __uint_as_float(w[j]);
+                        for (int j = 0; j < kChunk; ++j) v[j] = __uint_as_float(w[j / 8][j % 8]);
                     }
                     if (row < a.rows) {
-                        if (MODE == kDenseAddF32) {  // every old value is requested before the first is replaced
+                        if (MODE == kDenseAddF32) {
                             float* y = static_cast<float*>(a.out.y0) + (size_t)(m0 + c0) * a.out.ld0 + row;
-                            float old[8];
+                            float old[kChunk];
 #pragma unroll
-                            for (int j = 0; j < 8; ++j) old[j] = c0 + j < cnt ? y[(size_t)j * a.out.ld0] : 0.f;
+                            for (int j = 0; j < kChunk; ++j) old[j] = c0 + j < cnt ? y[(size_t)j * a.out.ld0] : 0.f;
 #pragma unroll
-                            for (int j = 0; j < 8; ++j)
+                            for (int j = 0; j < kChunk; ++j)
                                 if (c0 + j < cnt) y[(size_t)j * a.out.ld0] = old[j] + v[j];
-                        } else {
+                        } else if (MODE == kDenseStoreF32) {
+                            float* y = static_cast<float*>(a.out.y0) + (size_t)(m0 + c0) * a.out.ld0 + row;
 #pragma unroll
-                            for (int j = 0; j < 8; ++j)
-                                if (c0 + j < cnt) dense_store<MODE, bf16>(a.out, m0 + c0 + j, row, v[j]);
+                            for (int j = 0; j < kChunk; ++j)
+                                if (c0 + j < cnt) y[(size_t)j * a.out.ld0] = v[j];
+                        } else {
+                            const bool act = row >= a.out.split;
+                            const int ld = act ? a.out.ld1 : a.out.ld0;
+                            bf16* y = (act ? static_cast<bf16*>(a.out.y1) - a.out.split : static_cast<bf16*>(a.out.y0)) + (size_t)(m0 + c0) * ld + row;
+                            if (act) {
+#pragma unroll
+                                for (int j = 0; j < kChunk; ++j) v[j] = xielu_bf16(v[j], a.out.rising, a.out.falling);
+                            }
+#pragma unroll
+                            for (int j = 0; j < kChunk; ++j)
+                                if (c0 + j < cnt) y[(size_t)j * ld] = from_f32<bf16>(v[j]);
                         }
                     }
+                    __syncwarp();  // the next tensor-memory load needs the whole warp
                 }
             }
             tc_fence_before();
@@ -330,6 +343,14 @@ cudaError_t launch_bf16(const Launch& l, int mode, const DenseGemmArgs& a) {
 constexpr int kTile = 64, kStep = 32;
 
 template <int MODE>
+__device__ __forceinline__ void store_f32(const DenseOut& o, int token, int row, float v) {
+    float* y0 = static_cast<float*>(o.y0) + (size_t)token * o.ld0 + row;
+    if (MODE == kDenseAddF32) *y0 += v;
+    else if (MODE == kDenseStoreF32 || row < o.split) *y0 = v;
+    else static_cast<float*>(o.y1)[(size_t)token * o.ld1 + (row - o.split)] = xielu(v, o.rising, o.falling);
+}
+
+template <int MODE>
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const DenseGemmArgs a, DevDyn dyn) {
     __shared__ float xs[kTile][kStep + 1], ws[kTile][kStep + 1];
     pdl_trigger();
@@ -362,7 +383,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const DenseGemmArgs a, De
     for (int i = 0; i < 4; ++i)
 #pragma unroll
         for (int j = 0; j < 4; ++j)
-            if (m0 + ty + 16 * i < a.m && n0 + tx + 16 * j < a.rows) dense_store<MODE, float>(a.out, m0 + ty + 16 * i, n0 + tx + 16 * j, acc[i][j]);
+            if (m0 + ty + 16 * i < a.m && n0 + tx + 16 * j < a.rows) store_f32<MODE>(a.out, m0 + ty + 16 * i, n0 + tx + 16 * j, acc[i][j]);
 }
 
 cudaError_t launch_f32(const Launch& l, int mode, const DenseGemmArgs& a) {

@@ -2,11 +2,13 @@
 //
 // The activation row is staged once per CTA in fp32 (a decode step keeps all its activations in
 // fp32, so the only 16-bit operand is the stored weight) and, where the layer's norm is one
-// number, the norm is one factor per row that the epilogue applies.  A CTA owns a contiguous
-// range of rows; its eight warps form eight / KS row groups of KS warps that split the columns,
-// four rows at a time per group, so that every activation value read from shared memory feeds
-// four weights and each lane has eight 16-byte weight loads in flight.  Partial sums meet in
-// shared memory once per CTA and are added in warp order.
+// number, the norm is one factor per row that the epilogue applies.  One CTA per SM owns a
+// contiguous range of rows; its sixteen warps form 16 / KS row groups of KS warps that split the
+// columns.  A warp's work is a sequence of items of four rows x 256 columns, so that every
+// activation value read from shared memory feeds four weights; kDepth items are in flight in
+// registers (256 bytes a lane), across the end of a group of rows and, at the start, across the
+// wait for the launch in front, which the weights do not depend on.  Partial sums meet in shared
+// memory once per CTA and are added in warp order.
 #include <algorithm>
 
 #include "dense.h"
@@ -15,7 +17,7 @@ namespace smelt {
 
 namespace {
 
-constexpr int kThreads = 256, kWarps = 8, kRowsPerPass = 4, kChunkCols = 256;
+constexpr int kThreads = 512, kWarps = 16, kRowsPerPass = 4, kChunkCols = 256, kDepth = 4;
 
 __device__ __forceinline__ uint4 ld_stream(const uint4* p) {
     uint4 v;
@@ -34,28 +36,50 @@ __device__ __forceinline__ float dot8(const uint4& w, const float4& a, const flo
     return acc;
 }
 
+// The sums of four values over the warp; the lane gets the one of row 2 (lane bit 4) + (lane bit 3).
+__device__ __forceinline__ float sum_four_rows(const float (&v)[kRowsPerPass], int lane) {
+    const bool up = lane & 16, odd = lane & 8;
+    const float k0 = (up ? v[2] : v[0]) + __shfl_xor_sync(0xffffffffu, up ? v[0] : v[2], 16);
+    const float k1 = (up ? v[3] : v[1]) + __shfl_xor_sync(0xffffffffu, up ? v[1] : v[3], 16);
+    float k = (odd ? k1 : k0) + __shfl_xor_sync(0xffffffffu, odd ? k0 : k1, 8);
+#pragma unroll
+    for (int o = 4; o > 0; o >>= 1) k += __shfl_xor_sync(0xffffffffu, k, o);
+    return k;
+}
+
 template <int MODE>
-__global__ void __launch_bounds__(kThreads, 3) dense_matvec_kernel(const DenseMatvecArgs a, int rows_per_cta, int ks) {
+__global__ void __launch_bounds__(kThreads, 1) dense_matvec_kernel(const DenseMatvecArgs a, int rows_per_cta, int ks) {
     extern __shared__ __align__(16) float smem[];
     const int chunks = (a.cols + kChunkCols - 1) / kChunkCols;
     float* sx = smem;                          // [chunks][2][32][4]: a lane's eight values as two conflict-free halves
     float* part = smem + (size_t)chunks * kChunkCols;
     __shared__ float s_sum[kWarps];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int kid = warp % ks, group = warp / ks, groups = kWarps / ks;
+    const int kid = warp % ks, group = warp / ks, step = kWarps / ks * kRowsPerPass;
     const int r0 = blockIdx.x * rows_per_cta, r1 = min(a.rows, r0 + rows_per_cta);
     pdl_trigger();
 
-    // the first weights do not depend on the launch in front
-    uint4 first[kRowsPerPass];
-    const int c_first = kid * kChunkCols + lane * 8, base_first = r0 + group * kRowsPerPass;
+    struct Item { int row, chunk; };
+    auto next = [&](Item& it) {
+        it.chunk += ks;
+        if (it.chunk >= chunks) { it.chunk = kid; it.row += step; }
+    };
+    auto load = [&](const Item& it, uint4 (&dst)[kRowsPerPass]) {
+        const int col = it.chunk * kChunkCols + lane * 8;
+        const uint4* p = reinterpret_cast<const uint4*>(a.w + (size_t)it.row * a.cols + col);
+        const bool in = col < a.cols;
 #pragma unroll
-    for (int r = 0; r < kRowsPerPass; ++r)
-        first[r] = (base_first + r < r1 && c_first < a.cols) ? ld_stream(reinterpret_cast<const uint4*>(a.w + (size_t)(base_first + r) * a.cols + c_first)) : make_uint4(0, 0, 0, 0);
+        for (int r = 0; r < kRowsPerPass; ++r) dst[r] = in && it.row + r < r1 ? ld_stream(p + (size_t)r * (a.cols / 8)) : make_uint4(0, 0, 0, 0);
+    };
+    uint4 buf[kDepth][kRowsPerPass];
+    Item cur{r0 + group * kRowsPerPass, kid}, ahead = cur;
+#pragma unroll
+    for (int i = 0; i < kDepth; ++i) { load(ahead, buf[i]); next(ahead); }
 
     pdl_wait();
     if (dyn_skip(a.dyn)) return;
     float ss = 0.f;
+#pragma unroll 4
     for (int i = tid * 4; i < chunks * kChunkCols; i += kThreads * 4) {
         float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
         if (i < a.cols) v = *reinterpret_cast<const float4*>(a.xb && i >= a.ka ? a.xb + (i - a.ka) : a.xa + i);
@@ -76,29 +100,25 @@ __global__ void __launch_bounds__(kThreads, 3) dense_matvec_kernel(const DenseMa
         factor = a.gain * rsqrtf(tot / (float)a.width + a.eps);
     }
 
-    for (int base = base_first; base < r1; base += groups * kRowsPerPass) {
-        float acc[kRowsPerPass] = {0.f, 0.f, 0.f, 0.f};
-        const bf16* w0 = a.w + (size_t)base * a.cols + lane * 8;
-        const int left = r1 - base;
-#pragma unroll 2
-        for (int c = kid; c < chunks; c += ks) {
-            const int col = c * kChunkCols + lane * 8;
-            if (col < a.cols) {
-                uint4 wv[kRowsPerPass];
+    float acc[kRowsPerPass] = {0.f, 0.f, 0.f, 0.f};
+    while (cur.row < r1) {
 #pragma unroll
-                for (int r = 0; r < kRowsPerPass; ++r)
-                    wv[r] = base == base_first && c == kid ? first[r]
-                            : r < left                     ? ld_stream(reinterpret_cast<const uint4*>(w0 + (size_t)r * a.cols + c * kChunkCols))
-                                                           : make_uint4(0, 0, 0, 0);
-                const float4 xa = *reinterpret_cast<const float4*>(sx + c * kChunkCols + lane * 4);
-                const float4 xb = *reinterpret_cast<const float4*>(sx + c * kChunkCols + 128 + lane * 4);
+        for (int i = 0; i < kDepth; ++i) {
+            if (cur.row >= r1) break;
+            const float4 xa = *reinterpret_cast<const float4*>(sx + cur.chunk * kChunkCols + lane * 4);
+            const float4 xb = *reinterpret_cast<const float4*>(sx + cur.chunk * kChunkCols + 128 + lane * 4);
 #pragma unroll
-                for (int r = 0; r < kRowsPerPass; ++r) acc[r] = dot8(wv[r], xa, xb, acc[r]);
+            for (int r = 0; r < kRowsPerPass; ++r) acc[r] = dot8(buf[i][r], xa, xb, acc[r]);
+            load(ahead, buf[i]);
+            next(ahead);
+            if (cur.chunk + ks >= chunks) {  // the last columns of these rows
+                const float v = sum_four_rows(acc, lane);
+                const int row = cur.row + (lane >> 4) * 2 + ((lane >> 3) & 1);
+                if ((lane & 7) == 0 && row < r1) part[(size_t)(row - r0) * ks + kid] = v;
+                acc[0] = acc[1] = acc[2] = acc[3] = 0.f;
             }
+            next(cur);
         }
-#pragma unroll
-        for (int r = 0; r < kRowsPerPass; ++r) acc[r] = warp_sum(acc[r]);
-        if (lane < kRowsPerPass && lane < left) part[(size_t)(base - r0 + lane) * ks + kid] = lane == 0 ? acc[0] : lane == 1 ? acc[1] : lane == 2 ? acc[2] : acc[3];
     }
     __syncthreads();
     for (int i = tid; i < r1 - r0; i += kThreads) {
@@ -121,11 +141,9 @@ cudaError_t launch_dense_matvec(const Launch& l, int mode, DenseMatvecArgs a) {
     const int chunks = (a.cols + kChunkCols - 1) / kChunkCols;
     int ks = 1;
     while (ks < kWarps && ks * 2 <= chunks) ks *= 2;
-    const size_t x_bytes = (size_t)chunks * kChunkCols * sizeof(float), limit = 220 * 1024;
-    // as many CTAs as are resident at once, each with an equal share of the rows (at least one pass of its row groups)
-    int resident = (int)(limit / (x_bytes + 8192));
-    resident = resident < 1 ? 1 : resident > 3 ? 3 : resident;
-    int rows_per_cta = (a.rows + resident * sm - 1) / (resident * sm);
+    const size_t x_bytes = (size_t)chunks * kChunkCols * sizeof(float), limit = 225 * 1024;
+    // one CTA per SM with an equal share of the rows, at least what keeps its row groups busy
+    int rows_per_cta = (a.rows + sm - 1) / sm;
     rows_per_cta = std::max(rows_per_cta, std::min(kRowsPerPass * (kWarps / ks), 8));
     const int grid = (a.rows + rows_per_cta - 1) / rows_per_cta;
     const size_t smem = x_bytes + (size_t)rows_per_cta * ks * sizeof(float);

@@ -44,7 +44,12 @@ __device__ __forceinline__ float exp2_approx(float x) {
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
-__device__ __forceinline__ float cap_weight_of(const CapWeight& w, float dot) { return exp2_approx(w.top - __fdividef(w.span, exp2_approx(dot * w.rate) + 1.f)); }
+__device__ __forceinline__ float rcp_approx(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float cap_weight_of(const CapWeight& w, float dot) { return exp2_approx(fmaf(-w.span, rcp_approx(exp2_approx(dot * w.rate) + 1.f), w.top)); }
 
 // Shapes and softcaps the tensor-core kernels take.
 inline bool window_tiled(const WindowArgs& a) { return a.kp <= 256 && a.vp <= 256 && a.softcap > 0.f && a.softcap <= kMaxTiledCap; }

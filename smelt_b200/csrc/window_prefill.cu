@@ -1,12 +1,16 @@
 // Window + pooled-block attention of a prompt chunk on the tensor cores.
 //
 // The query heads that share a KV head are rows beside their positions: row = position * ratio +
-// head, 64 consecutive rows per CTA whatever the ratio, 16 per warp.  The CTA walks the blocks its
-// last position sees and then the window from its first position's start, 64 keys at a time; K and
-// V tiles are copied with cp.async into one of two swizzled buffers while the other is used.
+// head, 64 consecutive rows per CTA whatever the ratio.  The CTA walks the blocks its last
+// position sees and then the window from its first position's start, 64 keys at a time; K and V
+// tiles are copied with cp.async into one of two swizzled buffers while the other is used.  Eight
+// warps: four groups of sixteen rows times the two halves of a tile's keys, so that two CTAs give
+// an SM sixteen warps to hide each other's latencies; the halves' sums are added at the end.
 // S = Q K^T and O = P V with mma.sync m16n8k16 (bf16, fp32 accumulate), P as the sum of two bf16
 // values.  Weights need no running maximum (window.cuh), so nothing is rescaled.  Only tiles that
 // some row does not see in full are masked.
+#include <type_traits>
+
 #include "attention.cuh"
 #include "window.cuh"
 
@@ -14,7 +18,7 @@ namespace smelt {
 
 namespace {
 
-constexpr int kRows = 64, kKeys = 64, kThreads = 128;
+constexpr int kRows = 64, kKeys = 64, kHalf = kKeys / 2, kThreads = 256;
 
 __device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], uint32_t addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
@@ -30,8 +34,7 @@ template <int N> __device__ __forceinline__ uint32_t piece(int r, int c) { retur
 template <int D, int VD> __host__ __device__ constexpr size_t prefill_smem() { return (size_t)kRows * D * 2 + 2 * (size_t)kKeys * (D + VD) * 2; }
 
 template <int D, int VD>
-__global__ void __launch_bounds__(kThreads) window_prefill_kernel(const WindowArgs a, const CapWeight cw) {
-    constexpr bool kQInRegs = D <= 128;
+__global__ void __launch_bounds__(kThreads, D <= 128 && VD <= 128 ? 2 : 1) window_prefill_kernel(const WindowArgs a, const CapWeight cw) {
     constexpr int KS = D / 16;  // k steps of a score
     extern __shared__ __align__(128) unsigned char smem[];
     unsigned char* sQ = smem;
@@ -39,7 +42,7 @@ __global__ void __launch_bounds__(kThreads) window_prefill_kernel(const WindowAr
     unsigned char* sV = sK + 2 * kKeys * D * 2;      // [2]
     pdl_trigger();
     pdl_wait();
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, rw = warp & 3, kh = warp >> 2;
     const int kvh = blockIdx.y, ratio = a.heads / a.kv_heads, total = a.m * ratio;
     const int row0 = blockIdx.x * kRows, row_last = min(total, row0 + kRows) - 1;
     const uint32_t start = dyn_position(a.dyn), first = start + row0 / ratio, last = start + row_last / ratio;
@@ -50,18 +53,34 @@ __global__ void __launch_bounds__(kThreads) window_prefill_kernel(const WindowAr
     const bf16* K = static_cast<const bf16*>(a.k_cache) + kvh * head_rows * D;
     const bf16* V = static_cast<const bf16*>(a.v_cache) + kvh * head_rows * VD;
 
+    // a thread copies the same 16-byte column of every kThreads / (N / 8)-th row, a multiple of eight rows apart
+    auto copy_rows = [&](auto width, unsigned char* dst, const bf16* base, uint32_t row_first, bool contiguous, auto row_of) {
+        constexpr int N = decltype(width)::value, kStep = kThreads / (N / 8);
+        const int r0 = tid / (N / 8), c = tid % (N / 8);
+        dst += piece<N>(r0, c);
+        if (contiguous) {
+            const bf16* src = base + (size_t)(row_first + r0) * N + c * 8;
+#pragma unroll
+            for (int j = 0; j < kKeys / kStep; ++j) cp_async16(dst + j * kStep * N * 2, src + (size_t)j * kStep * N);
+        } else {
+#pragma unroll
+            for (int j = 0; j < kKeys / kStep; ++j) cp_async16(dst + j * kStep * N * 2, base + (size_t)row_of(r0 + j * kStep) * N + c * 8);
+        }
+    };
     auto issue_tile = [&](int tile, int buf) {
-        auto copy = [&](int r, int c, int n, unsigned char* dst, const bf16* base, uint32_t off) {
-            uint32_t row;
-            if (tile < pool_tiles) row = a.ring + min((uint32_t)(tile * kKeys + r), nb_last - 1u);
-            else {
-                row = lo_slot + min((uint32_t)((tile - pool_tiles) * kKeys + r), last - lo);
-                if (row >= a.ring) row -= a.ring;
-            }
-            cp_async16(dst + off, base + (size_t)row * n + c * 8);
+        const bool pooled = tile < pool_tiles;
+        const uint32_t off = (uint32_t)(pooled ? tile : tile - pool_tiles) * kKeys, count = pooled ? nb_last : last - lo + 1u;
+        uint32_t row_first = pooled ? a.ring + off : lo_slot + off;
+        if (!pooled && row_first >= a.ring) row_first -= a.ring;
+        const bool contiguous = off + kKeys <= count && (pooled || row_first + kKeys <= a.ring);
+        auto row_of = [&](int r) {  // keys past the end repeat the last one, their weights are zero
+            const uint32_t key = min(off + (uint32_t)r, count - 1u);
+            if (pooled) return a.ring + key;
+            const uint32_t s = lo_slot + key;
+            return s >= a.ring ? s - a.ring : s;
         };
-        for (int i = tid; i < kKeys * (D / 8); i += kThreads) { const int r = i / (D / 8), c = i % (D / 8); copy(r, c, D, sK + buf * kKeys * D * 2, K, piece<D>(r, c)); }
-        for (int i = tid; i < kKeys * (VD / 8); i += kThreads) { const int r = i / (VD / 8), c = i % (VD / 8); copy(r, c, VD, sV + buf * kKeys * VD * 2, V, piece<VD>(r, c)); }
+        copy_rows(std::integral_constant<int, D>(), sK + buf * kKeys * D * 2, K, row_first, contiguous, row_of);
+        copy_rows(std::integral_constant<int, VD>(), sV + buf * kKeys * VD * 2, V, row_first, contiguous, row_of);
         cp_async_commit();
     };
     {
@@ -73,14 +92,13 @@ __global__ void __launch_bounds__(kThreads) window_prefill_kernel(const WindowAr
     }
     issue_tile(0, 0);  // one group with the queries
 
-    // this thread's two rows: lane / 4 and lane / 4 + 8 of the warp's sixteen
-    const int my0 = min(row0 + warp * 16 + (lane >> 2), row_last), my1 = min(row0 + warp * 16 + (lane >> 2) + 8, row_last);
+    // this thread's two rows: lane / 4 and lane / 4 + 8 of the group's sixteen
+    const int my0 = min(row0 + rw * 16 + (lane >> 2), row_last), my1 = min(row0 + rw * 16 + (lane >> 2) + 8, row_last);
     const uint32_t i0 = start + my0 / ratio, i1 = start + my1 / ratio;
-    const uint32_t nb0 = min(visible_blocks(i0, a.window, a.pool), a.blocks), nb1 = min(visible_blocks(i1, a.window, a.pool), a.blocks);
-    const uint32_t lo0 = window_start(i0, a.window), lo1 = window_start(i1, a.window);
 
-    const uint32_t q_addr = smem_u32(sQ), q_row = warp * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, q_half = lane >> 4;
-    uint32_t qf[kQInRegs ? KS : 1][4];
+    const int l7 = lane & 7, b3 = (lane >> 3) & 1, b4 = lane >> 4;
+    const uint32_t q_addr = smem_u32(sQ) + (rw * 16 + l7 + b3 * 8) * (D * 2);
+    const uint32_t k_row = (kh * kHalf + l7 + b4 * 8) * (D * 2), v_row = (kh * kHalf + l7 + b3 * 8) * (VD * 2);
     float o[VD / 8][4], l0 = 0.f, l1 = 0.f;
 #pragma unroll
     for (int n = 0; n < VD / 8; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
@@ -91,49 +109,45 @@ __global__ void __launch_bounds__(kThreads) window_prefill_kernel(const WindowAr
         else cp_async_commit();
         cp_async_wait<1>();
         __syncthreads();
-        if (kQInRegs && tile == 0) {
-#pragma unroll
-            for (int k = 0; k < KS; ++k) ldsm_x4(qf[k], q_addr + piece<D>(q_row, 2 * k + q_half));
-        }
-        const uint32_t k_addr = smem_u32(sK + buf * kKeys * D * 2), v_addr = smem_u32(sV + buf * kKeys * VD * 2);
+        const uint32_t k_addr = smem_u32(sK + buf * kKeys * D * 2) + k_row, v_addr = smem_u32(sV + buf * kKeys * VD * 2) + v_row;
         const bool pooled = tile < pool_tiles;
-        const uint32_t base = pooled ? (uint32_t)tile * kKeys : lo + (uint32_t)(tile - pool_tiles) * kKeys;  // block or position of the tile's first key
-        const bool seen_in_full = pooled ? base + kKeys <= nb_first : base >= lo_last && base + kKeys - 1u <= first;
+        const uint32_t base = (pooled ? (uint32_t)tile * kKeys : lo + (uint32_t)(tile - pool_tiles) * kKeys) + kh * kHalf;  // block or position of this half's first key
+        const bool seen_in_full = pooled ? base + kHalf <= nb_first : base >= lo_last && base + kHalf - 1u <= first;
 
-        float s[kKeys / 8][4];
+        float s[kHalf / 8][4];
 #pragma unroll
-        for (int n = 0; n < kKeys / 8; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
+        for (int n = 0; n < kHalf / 8; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
 #pragma unroll
         for (int k = 0; k < KS; ++k) {
-            uint32_t qr[4];
-            if (!kQInRegs) ldsm_x4(qr, q_addr + piece<D>(q_row, 2 * k + q_half));
-            const uint32_t(&qv)[4] = kQInRegs ? qf[kQInRegs ? k : 0] : qr;
+            uint32_t qf[4];
+            ldsm_x4(qf, q_addr + (((2 * k + b4) ^ l7) << 4));
 #pragma unroll
-            for (int n = 0; n < kKeys / 16; ++n) {
+            for (int n = 0; n < kHalf / 16; ++n) {
                 uint32_t kf[4];
-                ldsm_x4(kf, k_addr + piece<D>(n * 16 + (lane & 7) + (lane >> 4) * 8, 2 * k + ((lane >> 3) & 1)));
-                mma16816_bf16(s[2 * n], qv[0], qv[1], qv[2], qv[3], kf[0], kf[1]);
-                mma16816_bf16(s[2 * n + 1], qv[0], qv[1], qv[2], qv[3], kf[2], kf[3]);
+                ldsm_x4(kf, k_addr + n * 16 * D * 2 + (((2 * k + b3) ^ l7) << 4));
+                mma16816_bf16(s[2 * n], qf[0], qf[1], qf[2], qf[3], kf[0], kf[1]);
+                mma16816_bf16(s[2 * n + 1], qf[0], qf[1], qf[2], qf[3], kf[2], kf[3]);
             }
         }
 #pragma unroll
-        for (int n = 0; n < kKeys / 8; ++n)
+        for (int n = 0; n < kHalf / 8; ++n)
 #pragma unroll
             for (int c = 0; c < 4; ++c) s[n][c] = cap_weight_of(cw, s[n][c]);
         if (!seen_in_full) {
+            const uint32_t end0 = pooled ? min(visible_blocks(i0, a.window, a.pool), a.blocks) : i0 + 1u, end1 = pooled ? min(visible_blocks(i1, a.window, a.pool), a.blocks) : i1 + 1u;
+            const uint32_t from0 = pooled ? 0u : window_start(i0, a.window), from1 = pooled ? 0u : window_start(i1, a.window);
 #pragma unroll
-            for (int n = 0; n < kKeys / 8; ++n)
+            for (int n = 0; n < kHalf / 8; ++n)
 #pragma unroll
                 for (int c = 0; c < 4; ++c) {
                     const uint32_t key = base + n * 8 + 2 * (lane & 3) + (c & 1);
-                    const bool seen = pooled ? key < (c < 2 ? nb0 : nb1) : key >= (c < 2 ? lo0 : lo1) && key <= (c < 2 ? i0 : i1);
-                    if (!seen) s[n][c] = 0.f;
+                    if (key < (c < 2 ? from0 : from1) || key >= (c < 2 ? end0 : end1)) s[n][c] = 0.f;
                 }
         }
 #pragma unroll
-        for (int n = 0; n < kKeys / 8; ++n) { l0 += s[n][0] + s[n][1]; l1 += s[n][2] + s[n][3]; }
+        for (int n = 0; n < kHalf / 8; ++n) { l0 += s[n][0] + s[n][1]; l1 += s[n][2] + s[n][3]; }
 #pragma unroll
-        for (int k = 0; k < kKeys / 16; ++k) {
+        for (int k = 0; k < kHalf / 16; ++k) {
             uint32_t hi[4], lo4[4];
 #pragma unroll
             for (int x = 0; x < 4; ++x) {  // (rows 0-7 | 8-15) of keys 0-7, then of keys 8-15
@@ -145,7 +159,7 @@ __global__ void __launch_bounds__(kThreads) window_prefill_kernel(const WindowAr
 #pragma unroll
             for (int n = 0; n < VD / 16; ++n) {
                 uint32_t vf[4];
-                ldsm_x4_trans(vf, v_addr + piece<VD>(k * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, 2 * n + (lane >> 4)));
+                ldsm_x4_trans(vf, v_addr + k * 16 * VD * 2 + (((2 * n + b4) ^ l7) << 4));
                 mma16816_bf16(o[2 * n], hi[0], hi[1], hi[2], hi[3], vf[0], vf[1]);
                 mma16816_bf16(o[2 * n + 1], hi[0], hi[1], hi[2], hi[3], vf[2], vf[3]);
                 mma16816_bf16(o[2 * n], lo4[0], lo4[1], lo4[2], lo4[3], vf[0], vf[1]);
@@ -157,22 +171,36 @@ __global__ void __launch_bounds__(kThreads) window_prefill_kernel(const WindowAr
     cp_async_wait<0>();
     l0 += __shfl_xor_sync(0xffffffffu, l0, 1); l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
     l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
+    // the second half's sums, in the tiles' memory
+    float4* so = reinterpret_cast<float4*>(sK) + (size_t)rw * (VD / 8) * 32 + lane;
+    float2* sl = reinterpret_cast<float2*>(sQ) + rw * 32 + lane;
+    if (kh == 1) {
+#pragma unroll
+        for (int n = 0; n < VD / 8; ++n) so[n * 32] = make_float4(o[n][0], o[n][1], o[n][2], o[n][3]);
+        *sl = make_float2(l0, l1);
+    }
+    __syncthreads();
+    if (kh == 1) return;
+    l0 += sl->x;
+    l1 += sl->y;
     const float f0 = 1.f / (l0 + cw.sink), f1 = 1.f / (l1 + cw.sink);
+    const int r0 = row0 + rw * 16 + (lane >> 2), r1 = r0 + 8;
+    auto out_row = [&](int row) { return static_cast<bf16*>(a.z) + (size_t)(row / ratio) * a.ldz + (kvh * ratio + row % ratio) * a.vdim; };
+    bf16 *z0 = out_row(min(r0, row_last)), *z1 = out_row(min(r1, row_last));
 #pragma unroll
-    for (int half = 0; half < 2; ++half) {
-        const int row = row0 + warp * 16 + (lane >> 2) + half * 8;
-        if (row >= total) continue;
-        const float f = half ? f1 : f0;
-        bf16* z = static_cast<bf16*>(a.z) + (size_t)(row / ratio) * a.ldz + (kvh * ratio + row % ratio) * a.vdim;
+    for (int n = 0; n < VD / 8; ++n) {
+        const int d = n * 8 + 2 * (lane & 3);
+        const float4 other = so[n * 32];
+        const float v[4] = {(o[n][0] + other.x) * f0, (o[n][1] + other.y) * f0, (o[n][2] + other.z) * f1, (o[n][3] + other.w) * f1};
 #pragma unroll
-        for (int n = 0; n < VD / 8; ++n) {
-            const int d = n * 8 + 2 * (lane & 3);
-            const float x = o[n][2 * half] * f, y = o[n][2 * half + 1] * f;
+        for (int half = 0; half < 2; ++half) {
+            if ((half ? r1 : r0) >= total) continue;
+            bf16* z = half ? z1 : z0;
             if (a.vdim % 2 == 0) {
-                if (d < a.vdim) *reinterpret_cast<uint32_t*>(z + d) = attn::TileElem<bf16>::pack(x, y);
+                if (d < a.vdim) *reinterpret_cast<uint32_t*>(z + d) = attn::TileElem<bf16>::pack(v[2 * half], v[2 * half + 1]);
             } else {
-                if (d < a.vdim) z[d] = from_f32<bf16>(x);
-                if (d + 1 < a.vdim) z[d + 1] = from_f32<bf16>(y);
+                if (d < a.vdim) z[d] = from_f32<bf16>(v[2 * half]);
+                if (d + 1 < a.vdim) z[d + 1] = from_f32<bf16>(v[2 * half + 1]);
             }
         }
     }
