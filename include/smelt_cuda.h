@@ -346,6 +346,13 @@ SMELT_CUDA_API smelt_status smelt_cuda_build_dense_prefill_table(smelt_cuda_ctx*
  * snapshots they are position-less state (a ring cannot be cut to a shorter length). */
 SMELT_CUDA_API smelt_status smelt_cuda_dense_cache_slots(const smelt_dense_desc* desc, int32_t* first_slot, int32_t* n_slots);
 
+/* What a package of the decoder lists: every slot its two tables bind except the weights, with its size (*n_slots: room in,
+ * count out; null arrays: count only), and the pipeline names of a table written without a context, newline separated. */
+SMELT_CUDA_API smelt_status smelt_cuda_dense_slots(const smelt_dense_desc* desc, const smelt_dense_layer* layers, uint32_t capacity, uint32_t max_chunk,
+                                                   int32_t* slots, uint64_t* bytes, int32_t* n_slots);
+SMELT_CUDA_API smelt_status smelt_cuda_dense_pipelines(const smelt_dense_desc* desc, const smelt_dense_layer* layers, uint32_t capacity, uint32_t max_chunk,
+                                                       int prefill, char* out, size_t out_bytes, size_t* needed_bytes);
+
 /* Typed launchers of those tables' kernels.  precision: SMELT_DENSE_BF16 or SMELT_DENSE_F32, the type T of a chunk's
  * activations and of the caches.  Weights are bf16, cols a multiple of 64 with zero padding.
  * mode: 0 y0 = fp32 product, 1 y0 += product (fp32), 2 rows below split to y0, the others through xIELU to y1, both in T

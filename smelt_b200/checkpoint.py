@@ -85,9 +85,11 @@ class TensorFile:
 
 @dataclass(frozen=True)
 class Architecture:
-    """parse: config dict -> configuration; decoder: (ctx, configuration, TensorFile, options) -> Decoder."""
+    """parse: config dict -> configuration; decoder: (ctx, configuration, TensorFile, options) -> Decoder;
+    write_package: (path, configuration, TensorFile, options), a ``.smeltpkg`` directory."""
     parse: Callable
     decoder: Callable
+    write_package: Callable
 
 
 _ARCHITECTURES: dict[str, Architecture] = {}
@@ -110,10 +112,22 @@ def architecture(config: dict) -> Architecture:
     return _ARCHITECTURES[name]
 
 
-def open_model(ctx, folder: str, **options):
-    """A decoder of the architecture the folder's ``config.json`` names.  Options: ``precision``
-    ("bfloat16" or "float32"), ``capacity`` (positions; 0 = all the model has), ``max_chunk``."""
+def read_model(folder: str):
+    """(architecture, configuration, tensors) of a model folder."""
     with open(os.path.join(folder, "config.json")) as f:
         config = json.load(f)
     arch = architecture(config)
-    return arch.decoder(ctx, arch.parse(config), TensorFile(read_safetensors(os.path.join(folder, "model.safetensors"))), **options)
+    return arch, arch.parse(config), TensorFile(read_safetensors(os.path.join(folder, "model.safetensors")))
+
+
+def open_model(ctx, folder: str, **options):
+    """A decoder of the architecture the folder's ``config.json`` names.  Options: ``precision``
+    ("bfloat16" or "float32"), ``capacity`` (positions; 0 = all the model has), ``max_chunk``."""
+    arch, config, tensors = read_model(folder)
+    return arch.decoder(ctx, config, tensors, **options)
+
+
+def convert(folder: str, path: str, **options) -> None:
+    """Writes a model folder as a ``.smeltpkg`` directory; options as in ``open_model``."""
+    arch, config, tensors = read_model(folder)
+    arch.write_package(path, config, tensors, **options)

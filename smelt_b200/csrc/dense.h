@@ -19,6 +19,12 @@ template <class T> __device__ __forceinline__ T from_f32(float v);
 template <> __device__ __forceinline__ float from_f32<float>(float v) { return v; }
 template <> __device__ __forceinline__ bf16 from_f32<bf16>(float v) { return __float2bfloat16_rn(v); }
 
+__device__ __forceinline__ float exp2_approx(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
 // xIELU: rising * z^2 + z / 2 for z > 0, falling * (exp(z) - 1 - z) + z / 2 otherwise, where
 // rising = softplus(p) and falling = 1 / 2 + softplus(q) of the layer's two stored numbers.
 __device__ __forceinline__ float xielu(float z, float rising, float falling) {

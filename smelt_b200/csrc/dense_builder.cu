@@ -5,7 +5,7 @@
 // matrices, [q; k; v; up] and [o | down], and a decoded token takes three launches per layer run:
 // norm + first matrix + xIELU, attention, second matrix + residual.
 #include <algorithm>
-#include <initializer_list>
+#include <map>
 #include <utility>
 #include <vector>
 
@@ -35,6 +35,8 @@ std::vector<Run> layer_runs(const smelt_dense_desc* d) {
     for (int l = d->loop_stop; l < d->layers; ++l) runs.push_back({l, false});
     return runs;
 }
+
+constexpr int kArgmaxChunk = 2048;
 
 int pad64(int n) { return (n + 63) / 64 * 64; }
 
@@ -68,62 +70,64 @@ const char* validate(const smelt_dense_desc* d, const smelt_dense_layer* layers,
     return nullptr;
 }
 
-smelt_status alloc_all(smelt_cuda_ctx* ctx, std::initializer_list<std::pair<int, size_t>> plan) {
-    for (auto& p : plan) {
-        smelt_status s = smelt_cuda_alloc_slot(ctx, p.first, p.second);
-        if (s) return s;
+using SlotPlan = std::vector<std::pair<int, size_t>>;
+
+// The slots one table binds, with their sizes.
+SlotPlan slot_plan(const smelt_dense_desc* d, const smelt_dense_layer* layers, uint32_t capacity, uint32_t max_chunk, bool prefill) {
+    const std::vector<Run> runs = layer_runs(d);
+    const size_t Wp = pad64(d->width), V = d->vocab, T = max_chunk, es = d->precision == SMELT_DENSE_F32 ? 4 : 2, parts = (V + kArgmaxChunk - 1) / kArgmaxChunk;
+    size_t u = 0, q = 0, z = 0;  // widest layer
+    for (int l = 0; l < d->layers; ++l) {
+        const LayerShape s = layer_shape(layers[l], capacity, max_chunk);
+        u = std::max(u, (size_t)s.qkv);
+        q = std::max(q, (size_t)layers[l].heads * s.kp);
+        z = std::max(z, (size_t)s.cols2);
     }
-    return SMELT_OK;
+    if (prefill)
+        return {{kDnPfX, T * Wp * 4}, {kDnPfX0, T * Wp * 4}, {kDnPfAct, T * 2 * Wp * es}, {kDnPfU, T * u * es}, {kDnPfQ, T * q * es}, {kDnPfZ, T * z * es},
+                {kLogits, T * V * 4}, {kArgmaxScratch, T * parts * 8}, {kArgmax, std::max<size_t>(T * 4, 8)}, {kTokenId, T * 4}, {kLogitRowsSlot, T * 4}};
+    SlotPlan plan = {{kHiddenA, Wp * 4}, {kHiddenB, Wp * 4}, {kDnEmbedding, Wp * 4}, {kDnU, u * 4}, {kDnQ, q * 4}, {kDnZ, z * 4},
+                     {kLogits, V * 4}, {kArgmax, 8}, {kTokenId, 4}, {kPosition, 8}, {kArgmaxScratch, parts * 8}};
+    for (size_t r = 0; r < runs.size(); ++r) {
+        const smelt_dense_layer& w = layers[runs[r].layer];
+        const LayerShape sh = layer_shape(w, capacity, max_chunk);
+        const size_t rows = (size_t)w.kv_heads * (sh.ring + sh.blocks);
+        plan.push_back({kKvBase + 2 * (int)r, rows * sh.kp * es});
+        plan.push_back({kKvBase + 2 * (int)r + 1, rows * sh.vp * es});
+    }
+    return plan;
 }
 
-struct Widest {
-    size_t u = 0, q = 0, z = 0;
-};
-
 smelt_status build(smelt_cuda_ctx* ctx, const smelt_dense_desc* d, const smelt_dense_layer* layers, uint32_t capacity, uint32_t max_chunk, bool prefill,
-                   smelt_dispatch_record* records, size_t* n_records) {
+                   smelt_dispatch_record* records, size_t* n_records, std::vector<std::string>* names = nullptr) {
     if (!d || !layers || !n_records) return SMELT_ERR_BAD_ARGUMENT;
     if (const char* why = validate(d, layers, capacity, max_chunk)) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, std::string("build_dense: ") + why);
     const std::vector<Run> runs = layer_runs(d);
-    const int W = d->width, Wp = pad64(W), V = d->vocab, chunk = 2048, parts = (V + chunk - 1) / chunk;
-    const size_t T = max_chunk, es = d->precision == SMELT_DENSE_F32 ? 4 : 2;
+    const int W = d->width, Wp = pad64(W), V = d->vocab, chunk = kArgmaxChunk, parts = (V + chunk - 1) / chunk;
+    const size_t es = d->precision == SMELT_DENSE_F32 ? 4 : 2;
     const std::string type = d->precision == SMELT_DENSE_F32 ? "_f32" : "_bf16";
-    Widest widest;
-    for (int l = 0; l < d->layers; ++l) {
-        const LayerShape s = layer_shape(layers[l], capacity, max_chunk);
-        widest.u = std::max(widest.u, (size_t)s.qkv);
-        widest.q = std::max(widest.q, (size_t)layers[l].heads * s.kp);
-        widest.z = std::max(widest.z, (size_t)s.cols2);
-    }
     Emitter e{ctx, records, records ? *n_records : 0};
     if (ctx) {
         if (!records) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, "build_dense: a context needs a record buffer (query the count with a null context)");
         if (cudaSetDevice(ctx->device) != cudaSuccess) return fail(ctx, SMELT_ERR_CUDA, "cudaSetDevice");
         if (!ctx->slots[kWeights].ptr) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, "build_dense: upload the weights image to slot 30 first");
-        smelt_status s = SMELT_OK;
+        if (kKvBase + 2 * runs.size() > ctx->slots.size()) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, "build_dense: too many layer runs for the slot table");
+        if (prefill && (!ctx->configured || !ctx->slots[kDnU].ptr)) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, "build_dense: build the decode table first");
+        for (auto& p : slot_plan(d, layers, capacity, max_chunk, prefill)) {
+            smelt_status s = smelt_cuda_alloc_slot(ctx, p.first, p.second);
+            if (s) return s;
+        }
         if (prefill) {
-            if (!ctx->configured || !ctx->slots[kDnU].ptr) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, "build_dense: build the decode table first");
-            s = alloc_all(ctx, {{kDnPfX, T * Wp * 4}, {kDnPfX0, T * Wp * 4}, {kDnPfAct, T * 2 * Wp * es}, {kDnPfU, T * widest.u * es}, {kDnPfQ, T * widest.q * es},
-                                {kDnPfZ, T * widest.z * es}, {kLogits, T * (size_t)V * 4}, {kArgmaxScratch, T * parts * 8}, {kArgmax, T * 4}, {kTokenId, T * 4}, {kLogitRowsSlot, T * 4}});
             e.base = (int)ctx->pipelines.size();
         } else {
-            if (kKvBase + 2 * runs.size() > ctx->slots.size()) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, "build_dense: too many layer runs for the slot table");
-            s = alloc_all(ctx, {{kHiddenA, (size_t)Wp * 4}, {kHiddenB, (size_t)Wp * 4}, {kDnEmbedding, (size_t)Wp * 4}, {kDnU, widest.u * 4}, {kDnQ, widest.q * 4}, {kDnZ, widest.z * 4},
-                                {kLogits, (size_t)V * 4}, {kArgmax, 8}, {kTokenId, 4}, {kPosition, 8}, {kArgmaxScratch, (size_t)parts * 8}});
-            for (size_t r = 0; r < runs.size() && !s; ++r) {
-                const smelt_dense_layer& w = layers[runs[r].layer];
-                const LayerShape sh = layer_shape(w, capacity, max_chunk);
-                const size_t rows = (size_t)w.kv_heads * (sh.ring + sh.blocks);
-                s = alloc_all(ctx, {{kKvBase + 2 * (int)r, rows * sh.kp * es}, {kKvBase + 2 * (int)r + 1, rows * sh.vp * es}});
-            }
             smelt_cuda_runtime_config cfg = {};
             cfg.token_id_slot = kTokenId; cfg.position_slot = kPosition; cfg.weights_slot = kWeights; cfg.argmax_slot = kArgmax;
             cfg.cur_slot = kHiddenA; cfg.alt_slot = kHiddenB; cfg.cache_seq_capacity = capacity; cfg.context_limit = capacity;
             cfg.vocab_size = (uint32_t)V; cfg.batch = 1;
-            if (!s) s = smelt_cuda_configure(ctx, &cfg);
+            smelt_status s = smelt_cuda_configure(ctx, &cfg);
+            if (s) return s;
             ctx->pipelines.clear();
         }
-        if (s) return s;
     }
 
     auto shaped = [&](const char* base, int cols, bool typed) { return std::string(base) + (typed ? type : "") + ":" + std::to_string(cols) + ":" + std::to_string(W); };
@@ -182,6 +186,10 @@ smelt_status build(smelt_cuda_ctx* ctx, const smelt_dense_desc* d, const smelt_d
         return fail(ctx, SMELT_ERR_BAD_ARGUMENT, "build_dense: record buffer too small");
     }
     *n_records = need;
+    if (names) {
+        names->assign(e.pipes.size(), std::string());
+        for (auto& kv : e.pipes) (*names)[kv.second - e.base] = kv.first;
+    }
     return e.status;
 }
 
@@ -201,5 +209,33 @@ extern "C" smelt_status smelt_cuda_dense_cache_slots(const smelt_dense_desc* des
     if (!desc || !first_slot || !n_slots || desc->loop_start < 0 || desc->loop_stop < desc->loop_start || desc->loop_stop > desc->layers || desc->loop_times < 0) return SMELT_ERR_BAD_ARGUMENT;
     *first_slot = kKvBase;
     *n_slots = 2 * (int32_t)layer_runs(desc).size();
+    return SMELT_OK;
+}
+
+extern "C" smelt_status smelt_cuda_dense_slots(const smelt_dense_desc* desc, const smelt_dense_layer* layers, uint32_t capacity, uint32_t max_chunk, int32_t* slots,
+                                               uint64_t* bytes, int32_t* n_slots) {
+    if (!desc || !layers || !n_slots || validate(desc, layers, capacity, max_chunk)) return SMELT_ERR_BAD_ARGUMENT;
+    std::map<int, size_t> all;
+    for (bool prefill : {false, true})
+        for (auto& p : slot_plan(desc, layers, capacity, max_chunk, prefill)) all[p.first] = std::max(all[p.first], p.second);
+    const int32_t room = *n_slots;
+    *n_slots = (int32_t)all.size();
+    if (!slots || !bytes) return SMELT_OK;
+    if (room < *n_slots) return SMELT_ERR_BAD_ARGUMENT;
+    for (auto& p : all) { *slots++ = p.first; *bytes++ = p.second; }
+    return SMELT_OK;
+}
+
+extern "C" smelt_status smelt_cuda_dense_pipelines(const smelt_dense_desc* desc, const smelt_dense_layer* layers, uint32_t capacity, uint32_t max_chunk, int prefill, char* out,
+                                                   size_t out_bytes, size_t* needed_bytes) {
+    if (!needed_bytes) return SMELT_ERR_BAD_ARGUMENT;
+    std::vector<std::string> names;
+    size_t n = 0;
+    smelt_status s = build(nullptr, desc, layers, capacity, max_chunk, prefill != 0, nullptr, &n, &names);
+    if (s) return s;
+    std::string joined;
+    for (auto& name : names) joined += name + "\n";
+    *needed_bytes = joined.size() + 1;
+    if (out && out_bytes >= joined.size() + 1) memcpy(out, joined.c_str(), joined.size() + 1);
     return SMELT_OK;
 }

@@ -26,9 +26,11 @@ namespace smelt {
 
 namespace {
 
-// xIELU for a bf16 result: the exponential's error (a few 2^-24 absolute near zero) is far below the result's rounding.
+// xIELU for a bf16 result, without a branch: the curve's two halves add, each zero on the other's
+// side.  The exponential's error (a few 2^-24 absolute near zero) is far below the result's rounding.
 __device__ __forceinline__ float xielu_bf16(float z, float rising, float falling) {
-    return fmaf(0.5f, z, z > 0.f ? rising * z * z : falling * (__expf(z) - 1.f - z));
+    const float pos = fmaxf(z, 0.f), neg = fminf(z, 0.f);
+    return fmaf(0.5f, z, fmaf(rising * pos, pos, falling * (exp2_approx(neg * 1.4426950408889634f) - 1.f - neg)));
 }
 
 // ── tcgen05 ─────────────────────────────────────────────────────────────────

@@ -170,7 +170,7 @@ struct Package {
     std::vector<std::string> pipelines;
     std::vector<SlotSpec> slots;
     int token_id_slot = -1, position_slot = -1, weights_slot = -1, key_base = -1, val_base = -1;
-    uint32_t vocab = 0, hidden = 0, layers = 0;
+    uint32_t vocab = 0, hidden = 0, layers = 0, static_capacity = 0;
     uint64_t weights_total = 0, weights_file = 0;
     uint32_t n_weight_entries = 0;
     std::vector<smelt_dispatch_record> table;
@@ -222,6 +222,7 @@ smelt_status load_package(const std::string& dir, Package& pk, std::string& err)
     pk.vocab = (uint32_t)v;
     if (get_int(config, "hiddenSize", &v)) pk.hidden = (uint32_t)v;
     if (get_int(config, "numLayers", &v)) pk.layers = (uint32_t)v;
+    if (get_int(config, "staticSeqCapacity", &v) && v > 0) pk.static_capacity = (uint32_t)v;
 
     const JVal* buffers = root.get("buffers");
     const JVal* slots = buffers ? buffers->get("slots") : nullptr;
@@ -229,8 +230,8 @@ smelt_status load_package(const std::string& dir, Package& pk, std::string& err)
     for (auto& s : slots->arr) {
         SlotSpec sp;
         int64_t idx = -1, bytes = 0;
-        if (!get_int(&s, "index", &idx) || !get_int(&s, "size_bytes", &bytes) || idx < 0 || idx >= 256 || bytes < 0) {
-            err = "manifest.json: a buffer slot lacks index / size_bytes, or its index is outside 0..255"; return SMELT_ERR_BAD_ARGUMENT;
+        if (!get_int(&s, "index", &idx) || !get_int(&s, "size_bytes", &bytes) || idx < 0 || idx >= kSlotCount || bytes < 0) {
+            err = "manifest.json: a buffer slot lacks index / size_bytes, or its index is outside the slot table"; return SMELT_ERR_BAD_ARGUMENT;
         }
         sp.index = (int)idx; sp.size_bytes = (uint64_t)bytes;
         if (const JVal* n = s.get("name")) sp.name = n->str;
@@ -395,6 +396,7 @@ smelt_status smelt_cuda_open_package(smelt_cuda_ctx* ctx, const char* package_di
     uint32_t capacity = options ? options->context_capacity : 0;
     for (const SlotSpec& sp : pk.slots)
         if (!capacity && is_kv_slot(sp) && sp.shape.size() >= 3 && sp.shape[1] > 0) capacity = (uint32_t)sp.shape[1];
+    if (!capacity) capacity = pk.static_capacity;  // window caches: no slot of one row per position
     if (!capacity) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, "open_package: no context capacity given and no KV cache slot to take it from");
     // weights.bin -> the weights slot (one device allocation; record offsets index it)
     {

@@ -39,11 +39,6 @@ inline CapWeight cap_weight(float scale, float softcap) {
     const double log2e = 1.4426950408889634, ref = softcap > 64.f ? softcap - 64.0 : 0.0;
     return CapWeight{(float)(2.0 * scale / softcap * log2e), (float)((softcap - ref) * log2e), (float)(2.0 * softcap * log2e), (float)exp(-ref)};
 }
-__device__ __forceinline__ float exp2_approx(float x) {
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
 __device__ __forceinline__ float rcp_approx(float x) {
     float y;
     asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));

@@ -1,11 +1,12 @@
 // Window + pooled-block attention of a prompt chunk on the tensor cores.
 //
 // The query heads that share a KV head are rows beside their positions: row = position * ratio +
-// head, 64 consecutive rows per CTA whatever the ratio.  The CTA walks the blocks its last
+// head, 16 RG consecutive rows per CTA whatever the ratio.  The CTA walks the blocks its last
 // position sees and then the window from its first position's start, 64 keys at a time; K and V
 // tiles are copied with cp.async into one of two swizzled buffers while the other is used.  Eight
-// warps: four groups of sixteen rows times the two halves of a tile's keys, so that two CTAs give
-// an SM sixteen warps to hide each other's latencies; the halves' sums are added at the end.
+// warps: RG groups of sixteen rows times 8 / RG parts of a tile's keys, so that two CTAs give an SM
+// sixteen warps to hide each other's latencies; the parts' sums are added at the end.  RG is 4, or 2
+// where that leaves SMs without a CTA (the kernel is bound by the latency of one CTA's walk).
 // S = Q K^T and O = P V with mma.sync m16n8k16 (bf16, fp32 accumulate), P as the sum of two bf16
 // values.  Weights need no running maximum (window.cuh), so nothing is rescaled.  Only tiles that
 // some row does not see in full are masked.
@@ -18,7 +19,7 @@ namespace smelt {
 
 namespace {
 
-constexpr int kRows = 64, kKeys = 64, kHalf = kKeys / 2, kThreads = 256;
+constexpr int kKeys = 64, kThreads = 256;
 
 __device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], uint32_t addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
@@ -31,18 +32,19 @@ __device__ __forceinline__ void ldsm_x4_trans(uint32_t (&r)[4], uint32_t addr) {
 // neighbouring rows fall into different banks.
 template <int N> __device__ __forceinline__ uint32_t piece(int r, int c) { return (uint32_t)(r * (N * 2) + ((c ^ (r & 7)) << 4)); }
 
-template <int D, int VD> __host__ __device__ constexpr size_t prefill_smem() { return (size_t)kRows * D * 2 + 2 * (size_t)kKeys * (D + VD) * 2; }
+template <int D, int VD, int RG> __host__ __device__ constexpr size_t prefill_smem() { return (size_t)16 * RG * D * 2 + 2 * (size_t)kKeys * (D + VD) * 2; }
 
-template <int D, int VD>
+template <int D, int VD, int RG>
 __global__ void __launch_bounds__(kThreads, D <= 128 && VD <= 128 ? 2 : 1) window_prefill_kernel(const WindowArgs a, const CapWeight cw) {
     constexpr int KS = D / 16;  // k steps of a score
+    constexpr int kRows = 16 * RG, kParts = 8 / RG, kPart = kKeys / kParts;
     extern __shared__ __align__(128) unsigned char smem[];
     unsigned char* sQ = smem;
     unsigned char* sK = sQ + kRows * D * 2;          // [2]
     unsigned char* sV = sK + 2 * kKeys * D * 2;      // [2]
     pdl_trigger();
     pdl_wait();
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, rw = warp & 3, kh = warp >> 2;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, rw = warp % RG, kp = warp / RG;
     const int kvh = blockIdx.y, ratio = a.heads / a.kv_heads, total = a.m * ratio;
     const int row0 = blockIdx.x * kRows, row_last = min(total, row0 + kRows) - 1;
     const uint32_t start = dyn_position(a.dyn), first = start + row0 / ratio, last = start + row_last / ratio;
@@ -98,7 +100,7 @@ __global__ void __launch_bounds__(kThreads, D <= 128 && VD <= 128 ? 2 : 1) windo
 
     const int l7 = lane & 7, b3 = (lane >> 3) & 1, b4 = lane >> 4;
     const uint32_t q_addr = smem_u32(sQ) + (rw * 16 + l7 + b3 * 8) * (D * 2);
-    const uint32_t k_row = (kh * kHalf + l7 + b4 * 8) * (D * 2), v_row = (kh * kHalf + l7 + b3 * 8) * (VD * 2);
+    const uint32_t k_row = (kp * kPart + l7 + b4 * 8) * (D * 2), v_row = (kp * kPart + l7 + b3 * 8) * (VD * 2);
     float o[VD / 8][4], l0 = 0.f, l1 = 0.f;
 #pragma unroll
     for (int n = 0; n < VD / 8; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
@@ -111,18 +113,18 @@ __global__ void __launch_bounds__(kThreads, D <= 128 && VD <= 128 ? 2 : 1) windo
         __syncthreads();
         const uint32_t k_addr = smem_u32(sK + buf * kKeys * D * 2) + k_row, v_addr = smem_u32(sV + buf * kKeys * VD * 2) + v_row;
         const bool pooled = tile < pool_tiles;
-        const uint32_t base = (pooled ? (uint32_t)tile * kKeys : lo + (uint32_t)(tile - pool_tiles) * kKeys) + kh * kHalf;  // block or position of this half's first key
-        const bool seen_in_full = pooled ? base + kHalf <= nb_first : base >= lo_last && base + kHalf - 1u <= first;
+        const uint32_t base = (pooled ? (uint32_t)tile * kKeys : lo + (uint32_t)(tile - pool_tiles) * kKeys) + kp * kPart;  // block or position of this part's first key
+        const bool seen_in_full = pooled ? base + kPart <= nb_first : base >= lo_last && base + kPart - 1u <= first;
 
-        float s[kHalf / 8][4];
+        float s[kPart / 8][4];
 #pragma unroll
-        for (int n = 0; n < kHalf / 8; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
+        for (int n = 0; n < kPart / 8; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
 #pragma unroll
         for (int k = 0; k < KS; ++k) {
             uint32_t qf[4];
             ldsm_x4(qf, q_addr + (((2 * k + b4) ^ l7) << 4));
 #pragma unroll
-            for (int n = 0; n < kHalf / 16; ++n) {
+            for (int n = 0; n < kPart / 16; ++n) {
                 uint32_t kf[4];
                 ldsm_x4(kf, k_addr + n * 16 * D * 2 + (((2 * k + b3) ^ l7) << 4));
                 mma16816_bf16(s[2 * n], qf[0], qf[1], qf[2], qf[3], kf[0], kf[1]);
@@ -130,14 +132,14 @@ __global__ void __launch_bounds__(kThreads, D <= 128 && VD <= 128 ? 2 : 1) windo
             }
         }
 #pragma unroll
-        for (int n = 0; n < kHalf / 8; ++n)
+        for (int n = 0; n < kPart / 8; ++n)
 #pragma unroll
             for (int c = 0; c < 4; ++c) s[n][c] = cap_weight_of(cw, s[n][c]);
         if (!seen_in_full) {
             const uint32_t end0 = pooled ? min(visible_blocks(i0, a.window, a.pool), a.blocks) : i0 + 1u, end1 = pooled ? min(visible_blocks(i1, a.window, a.pool), a.blocks) : i1 + 1u;
             const uint32_t from0 = pooled ? 0u : window_start(i0, a.window), from1 = pooled ? 0u : window_start(i1, a.window);
 #pragma unroll
-            for (int n = 0; n < kHalf / 8; ++n)
+            for (int n = 0; n < kPart / 8; ++n)
 #pragma unroll
                 for (int c = 0; c < 4; ++c) {
                     const uint32_t key = base + n * 8 + 2 * (lane & 3) + (c & 1);
@@ -145,9 +147,9 @@ __global__ void __launch_bounds__(kThreads, D <= 128 && VD <= 128 ? 2 : 1) windo
                 }
         }
 #pragma unroll
-        for (int n = 0; n < kHalf / 8; ++n) { l0 += s[n][0] + s[n][1]; l1 += s[n][2] + s[n][3]; }
+        for (int n = 0; n < kPart / 8; ++n) { l0 += s[n][0] + s[n][1]; l1 += s[n][2] + s[n][3]; }
 #pragma unroll
-        for (int k = 0; k < kHalf / 16; ++k) {
+        for (int k = 0; k < kPart / 16; ++k) {
             uint32_t hi[4], lo4[4];
 #pragma unroll
             for (int x = 0; x < 4; ++x) {  // (rows 0-7 | 8-15) of keys 0-7, then of keys 8-15
@@ -171,18 +173,23 @@ __global__ void __launch_bounds__(kThreads, D <= 128 && VD <= 128 ? 2 : 1) windo
     cp_async_wait<0>();
     l0 += __shfl_xor_sync(0xffffffffu, l0, 1); l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
     l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
-    // the second half's sums, in the tiles' memory
+    // the other parts' sums, in the tiles' memory
+    static_assert((size_t)(kParts - 1) * RG * (VD / 8) * 512 <= 2 * (size_t)kKeys * (D + VD) * 2 && (size_t)(kParts - 1) * RG * 256 <= (size_t)kRows * D * 2, "the sums fit where the tiles were");
     float4* so = reinterpret_cast<float4*>(sK) + (size_t)rw * (VD / 8) * 32 + lane;
     float2* sl = reinterpret_cast<float2*>(sQ) + rw * 32 + lane;
-    if (kh == 1) {
+    constexpr int kSo = RG * (VD / 8) * 32, kSl = RG * 32;  // per part
+    if (kp > 0) {
 #pragma unroll
-        for (int n = 0; n < VD / 8; ++n) so[n * 32] = make_float4(o[n][0], o[n][1], o[n][2], o[n][3]);
-        *sl = make_float2(l0, l1);
+        for (int n = 0; n < VD / 8; ++n) so[(kp - 1) * kSo + n * 32] = make_float4(o[n][0], o[n][1], o[n][2], o[n][3]);
+        sl[(kp - 1) * kSl] = make_float2(l0, l1);
     }
     __syncthreads();
-    if (kh == 1) return;
-    l0 += sl->x;
-    l1 += sl->y;
+    if (kp > 0) return;
+#pragma unroll
+    for (int p = 0; p < kParts - 1; ++p) {
+        l0 += sl[p * kSl].x;
+        l1 += sl[p * kSl].y;
+    }
     const float f0 = 1.f / (l0 + cw.sink), f1 = 1.f / (l1 + cw.sink);
     const int r0 = row0 + rw * 16 + (lane >> 2), r1 = r0 + 8;
     auto out_row = [&](int row) { return static_cast<bf16*>(a.z) + (size_t)(row / ratio) * a.ldz + (kvh * ratio + row % ratio) * a.vdim; };
@@ -190,8 +197,12 @@ __global__ void __launch_bounds__(kThreads, D <= 128 && VD <= 128 ? 2 : 1) windo
 #pragma unroll
     for (int n = 0; n < VD / 8; ++n) {
         const int d = n * 8 + 2 * (lane & 3);
-        const float4 other = so[n * 32];
-        const float v[4] = {(o[n][0] + other.x) * f0, (o[n][1] + other.y) * f0, (o[n][2] + other.z) * f1, (o[n][3] + other.w) * f1};
+#pragma unroll
+        for (int p = 0; p < kParts - 1; ++p) {
+            const float4 other = so[p * kSo + n * 32];
+            o[n][0] += other.x; o[n][1] += other.y; o[n][2] += other.z; o[n][3] += other.w;
+        }
+        const float v[4] = {o[n][0] * f0, o[n][1] * f0, o[n][2] * f1, o[n][3] * f1};
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
             if ((half ? r1 : r0) >= total) continue;
@@ -206,18 +217,27 @@ __global__ void __launch_bounds__(kThreads, D <= 128 && VD <= 128 ? 2 : 1) windo
     }
 }
 
-template <int D, int VD>
+template <int D, int VD, int RG>
 cudaError_t launch_t(const Launch& l, const WindowArgs& a) {
-    const dim3 grid((unsigned)(((size_t)a.m * (a.heads / a.kv_heads) + kRows - 1) / kRows), a.kv_heads);
-    return launch_chained(l, window_prefill_kernel<D, VD>, grid, dim3(kThreads), prefill_smem<D, VD>(), a, cap_weight(a.scale, a.softcap));
+    const dim3 grid((unsigned)(((size_t)a.m * (a.heads / a.kv_heads) + 16 * RG - 1) / (16 * RG)), a.kv_heads);
+    return launch_chained(l, window_prefill_kernel<D, VD, RG>, grid, dim3(kThreads), prefill_smem<D, VD, RG>(), a, cap_weight(a.scale, a.softcap));
+}
+
+template <int D, int VD>
+cudaError_t launch_rows(const Launch& l, const WindowArgs& a) {
+    if constexpr (D <= 128 && VD <= 128) {
+        const size_t ctas = ((size_t)a.m * (a.heads / a.kv_heads) + 63) / 64 * a.kv_heads;
+        if (ctas <= (size_t)(a.sm_count > 0 ? a.sm_count : 148)) return launch_t<D, VD, 2>(l, a);
+    }
+    return launch_t<D, VD, 4>(l, a);
 }
 
 template <int D>
 cudaError_t launch_values(const Launch& l, const WindowArgs& a) {
     switch (a.vp) {
-        case 64: return launch_t<D, 64>(l, a);
-        case 128: return launch_t<D, 128>(l, a);
-        default: return launch_t<D, 256>(l, a);
+        case 64: return launch_rows<D, 64>(l, a);
+        case 128: return launch_rows<D, 128>(l, a);
+        default: return launch_rows<D, 256>(l, a);
     }
 }
 

@@ -654,6 +654,10 @@ def write_package(path: str, cfg: DecoderConfig, image: np.ndarray, desc: capi.D
         "slotLayout": {"convStateBaseSlot": -1, "recStateBaseSlot": -1, "keyCacheBaseSlot": KV_BASE_SLOT, "valCacheBaseSlot": KV_BASE_SLOT + cfg.layers,
                        "ropeCosSlot": -1, "ropeSinSlot": -1, "ropeTablePairs": [], "tokenIdSlot": 33, "positionSlot": 34, "weightsSlot": WEIGHTS_SLOT},
     }
+    _write_package_files(path, manifest, image, table, prefill_table)
+
+
+def _write_package_files(path: str, manifest: dict, image: np.ndarray, table, prefill_table) -> None:
     with open(os.path.join(path, "manifest.json"), "w") as f:
         json.dump(manifest, f, sort_keys=True)
     np.asarray(image, np.uint8).tofile(os.path.join(path, "weights.bin"))
@@ -662,6 +666,56 @@ def write_package(path: str, cfg: DecoderConfig, image: np.ndarray, desc: capi.D
     if prefill_table is not None:
         with open(os.path.join(path, "prefill_dispatches.bin"), "wb") as f:
             f.write(bytes(prefill_table))
+
+
+def write_dense_package(path: str, name: str, image: np.ndarray, desc: capi.DenseDesc, layers, entries: list, capacity: int, precision: str = "bfloat16",
+                        max_chunk: int = 512) -> None:
+    """Writes a decoder with dense 16-bit weights as a ``.smeltpkg`` that the package reader opens: both record
+    tables, their pipelines and slots, the weights image.  entries: (tensor name, offset, size in bytes, shape)."""
+    lib = capi.load()
+    os.makedirs(path, exist_ok=True)
+    desc.precision = DenseDecoder.PRECISIONS[precision]
+    chunk = int(min(max_chunk, capacity))
+
+    def text(prefill: int) -> list[str]:
+        need = C.c_size_t(0)
+        lib.smelt_cuda_dense_pipelines(C.byref(desc), layers, capacity, chunk, prefill, None, C.c_size_t(0), C.byref(need))
+        buf = C.create_string_buffer(need.value)
+        lib.smelt_cuda_dense_pipelines(C.byref(desc), layers, capacity, chunk, prefill, buf, C.c_size_t(need.value), C.byref(need))
+        return [p for p in buf.value.decode().split("\n") if p]
+
+    def table(build):
+        n = C.c_size_t(0)
+        st = build(None, C.byref(desc), layers, capacity, chunk, None, C.byref(n))
+        out = (capi.DispatchRecord * n.value)()
+        st = st or build(None, C.byref(desc), layers, capacity, chunk, out, C.byref(n))
+        if st != 0:
+            raise capi.SmeltError(st, "build_dense (dry run) failed")
+        return out
+
+    decode, prefill = table(lib.smelt_cuda_build_dense_decoder), table(lib.smelt_cuda_build_dense_prefill_table)
+    pipelines = text(0)
+    for r in prefill:  # the dry run numbers its pipelines from 0: they follow the decode table's in the manifest
+        if r.op_kind == 0:
+            r.pipeline += len(pipelines)
+    pipelines += text(1)
+    n = C.c_int32(0)
+    lib.smelt_cuda_dense_slots(C.byref(desc), layers, capacity, chunk, None, None, C.byref(n))
+    index, size = (C.c_int32 * n.value)(), (C.c_uint64 * n.value)()
+    lib.smelt_cuda_dense_slots(C.byref(desc), layers, capacity, chunk, index, size, C.byref(n))
+    slots = [{"index": int(i), "name": f"windowCache_{i - KV_BASE_SLOT}" if i >= KV_BASE_SLOT else f"slot_{i}", "size_bytes": int(b), "dtype": "raw", "shape": [int(b)],
+              "category": "state" if i >= KV_BASE_SLOT else "activation"} for i, b in zip(index, size)]
+    slots.append({"index": WEIGHTS_SLOT, "name": "weights", "size_bytes": 0, "dtype": "raw", "shape": [], "category": "weight"})
+    manifest = {
+        "version": 1, "kind": "text-generation", "architecture": "text-generation", "modelName": name,
+        "config": {"hiddenSize": desc.width, "numLayers": desc.layers, "vocabSize": desc.vocab, "staticSeqCapacity": int(capacity)},
+        "checksums": {}, "device": {},
+        "weights": {"total_bytes": int(image.nbytes), "entries": [{"name": e[0], "offset": int(e[1]), "size_bytes": int(e[2]), "shape": list(e[3]), "dtype": "bf16"} for e in entries]},
+        "buffers": {"slots": slots}, "pipelines": pipelines,
+        "slotLayout": {"convStateBaseSlot": -1, "recStateBaseSlot": -1, "keyCacheBaseSlot": -1, "valCacheBaseSlot": -1, "ropeCosSlot": -1, "ropeSinSlot": -1, "ropeTablePairs": [],
+                       "tokenIdSlot": 33, "positionSlot": 34, "weightsSlot": WEIGHTS_SLOT},
+    }
+    _write_package_files(path, manifest, image, decode, prefill)
 
 
 class PackageSession:

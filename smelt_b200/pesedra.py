@@ -113,8 +113,8 @@ def build_image(c: Config, tensors: checkpoint.TensorFile):
     [q; k; v; up], its output projections as one matrix [o | down]."""
     img = package.WeightsImage()
     layers = (capi.DenseLayer * len(c.layers))()
-    get = lambda name: tensors.bf16(name, *shapes[name])
     shapes = tensor_shapes(c)
+    get = lambda name: tensors.bf16(name, *shapes[name])
     for i, m in enumerate(c.layers):
         p, w = f"l{i}", layers[i]
         w.heads, w.kv_heads, w.dim, w.vdim, w.window, w.pool, w.ff = m.heads, m.kv_heads, m.dim, m.vdim, m.window, m.pool, m.ff
@@ -142,4 +142,18 @@ def decoder(ctx, c: Config, tensors: checkpoint.TensorFile, precision: str = "bf
     return package.DenseDecoder(ctx, image, desc, layers, capacity=min(capacity or c.max_positions, c.max_positions), precision=precision, max_chunk=max_chunk)
 
 
-checkpoint.register("Pesedra", checkpoint.Architecture(parse, decoder))
+def write_package(path: str, c: Config, tensors: checkpoint.TensorFile, precision: str = "bfloat16", capacity: int = 0, max_chunk: int = 512) -> None:
+    """The model as a ``.smeltpkg`` directory."""
+    image, desc, layers = build_image(c, tensors)
+    pad = lambda n: -(-n // 64) * 64
+    entries = [("embed", desc.embedding, c.vocab, c.width), ("pos", desc.positions, c.max_positions, c.width), ("head", desc.lm_head, c.vocab, pad(c.width))]
+    if c.loop[1] > c.loop[0]:
+        entries.append(("loop.in", desc.loop_in, c.width, 2 * pad(c.width)))
+    for i, (m, w) in enumerate(zip(c.layers, layers)):
+        entries += [(f"l{i}.in", w.in_proj, m.qkv + m.ff, pad(c.width)), (f"l{i}.out", w.out_proj, c.width, pad(m.heads * m.vdim + m.ff)),
+                    (f"l{i}.q.norm", w.q_norm, 1, m.dim), (f"l{i}.k.norm", w.k_norm, 1, m.dim)]
+    package.write_dense_package(path, "pesedra", image, desc, layers, [(n, off, rows * cols * 2, (rows, cols)) for n, off, rows, cols in entries],
+                                min(capacity or c.max_positions, c.max_positions), precision, max_chunk)
+
+
+checkpoint.register("Pesedra", checkpoint.Architecture(parse, decoder, write_package))

@@ -228,6 +228,19 @@ def test_window_attention(ctx, geometry, precision, cut):
     assert worst(got, want) < 2e-5 if precision == "float32" else worst_row(got, want) < 0.015
 
 
+@pytest.mark.parametrize("dim,vdim", [(64, 128), (128, 64), (128, 128)])
+def test_long_chunk(ctx, dim, vdim):
+    """Enough CTAs that every SM has one: the other cut of rows and keys over a CTA's warps."""
+    w = Window(ctx, "bfloat16", 24, 6, dim, vdim, 150, 10, 2.0 / np.sqrt(dim), 12.0, positions=620, chunk=512)
+    u = np.random.default_rng(dim).standard_normal((600, 24 * dim + 6 * (dim + vdim)))
+    got = np.concatenate([w.feed(u[:88]), w.feed(u[88:])])
+    rows = list(range(0, 600, 7)) + [599]
+    q, k, v = w.split(seen_as(u, "bfloat16"))
+    q, k = (seen_as(ref.head_rms_norm(x, n, w.desc.eps), "bfloat16") for x, n in ((q, w.qn), (k, w.kn)))
+    want = np.concatenate([ref.window_pool_attention(q[i:i + 1], k, v, i, w.desc.scale, 12.0, 150, 10) for i in rows])
+    assert worst_row(got[rows], want) < 0.015
+
+
 @pytest.mark.parametrize("precision", PRECISIONS)
 @pytest.mark.parametrize("softcap", [0.0, 5.0, 80.0, 200.0])
 def test_softcaps(ctx, precision, softcap):
@@ -442,3 +455,36 @@ def test_trace_run_program(ctx, tmp_path, precision):
     for i, want in ((0, la[[0, 76]]), (1, la[[97]]), (3, la[[99]]), (4, lb[[29]])):
         assert worst_row(read(i), want) < LIMIT[precision]
     assert not (out / "2.f32").exists()
+
+
+@pytest.mark.parametrize("precision", PRECISIONS)
+def test_package_runs_as_the_model_does(ctx, tmp_path, precision):
+    cfg = cases.MIXED
+    arch, t = checkpoint.architecture(cfg), cases.tensors(cfg)
+    arch.write_package(str(tmp_path / "m.smeltpkg"), arch.parse(cfg), checkpoint.TensorFile(cases.stored(t)), precision=precision, max_chunk=64)
+    dec, _ = open_decoder(ctx, "mixed", precision)
+    prompt = cases.tokens(cfg, 90, 21)
+    want = dec.generate(prompt, 30)[:, 0]
+    other = capi.Context(0)
+    session = package.PackageSession(other, str(tmp_path / "m.smeltpkg"))
+    got = [session.prefill(prompt, chunk=64)]
+    for i in range(9):
+        got.append(session.decode_step(got[-1], 90 + i))
+    session.build_graph()
+    for i in range(9, 29):
+        got.append(session.graph_step(got[-1], 90 + i))
+    np.testing.assert_array_equal(got, want)
+    with pytest.raises(capi.SmeltError):
+        session.prefill(prompt, chunk=90)  # more than the tables were compiled for
+    other.close()
+
+
+def test_generate_command(tmp_path, capsys, ctx):
+    from smelt_b200 import generate
+
+    cfg = cases.ODD
+    (tmp_path / "config.json").write_text(json.dumps(cfg))
+    checkpoint.write_safetensors(str(tmp_path / "model.safetensors"), cases.stored(cases.tensors(cfg)))
+    dec, _ = open_decoder(ctx, "odd", "float32")
+    assert generate.main(["--model", str(tmp_path), "--prompt", "5,6,7,8", "--tokens", "12", "--dtype", "float32"]) == 0
+    assert [int(x) for x in capsys.readouterr().out.split()] == dec.generate([5, 6, 7, 8], 12)[:, 0].tolist()

@@ -8,7 +8,7 @@ import pytest
 
 import pesedra_cases as cases
 from oracle import pesedra as ref
-from smelt_b200 import capi, checkpoint, pesedra, trace_run
+from smelt_b200 import capi, checkpoint, generate, package, pesedra, trace_run
 
 
 # ── the restatement ─────────────────────────────────────────────────────────
@@ -164,6 +164,22 @@ def test_dense_kernel_names_are_bound():
     assert lib.smelt_cuda_pipeline_supported(b"smelt_window_decode_fp8") == 0
 
 
+@pytest.mark.parametrize("name", cases.ALL)
+def test_package_of_the_model_validates(tmp_path, name):
+    cfg, folder, out = cases.ALL[name], tmp_path / "model", tmp_path / "x.smeltpkg"
+    folder.mkdir()
+    (folder / "config.json").write_text(json.dumps(cfg))
+    checkpoint.write_safetensors(str(folder / "model.safetensors"), cases.stored(cases.tensors(cfg)))
+    checkpoint.convert(str(folder), str(out), max_chunk=64)
+    st, info, err = package.inspect_package(str(out))
+    assert st == 0, err
+    runs = len(pesedra.parse(cfg).runs())
+    assert info.vocab_size == cfg["vocab"] and info.n_prefill_records > 6 * runs and info.n_records > 3 * runs
+    manifest = json.loads((out / "manifest.json").read_text())
+    assert sum(s["category"] == "state" for s in manifest["buffers"]["slots"]) == 2 * runs
+    assert all(e["offset"] % 128 == 0 for e in manifest["weights"]["entries"])
+
+
 # ── trace replay ────────────────────────────────────────────────────────────
 class FakeDecoder:
     def __init__(self):
@@ -184,3 +200,8 @@ def test_replay_follows_one_sequence_at_a_time():
     assert d.calls == [([5, 6, 7], 0, [0, 2]), ([8], 3, []), ([9], 0, [0])]
     with pytest.raises(ValueError, match="live"):
         r.step([{"id": "c", "tokens": [1], "want": []}], [])
+
+
+def test_prompt_ids(tmp_path):
+    (tmp_path / "ids").write_text("4, 5\n6")
+    assert generate.parse_ids("1,2,3") == [1, 2, 3] and generate.parse_ids(f"@{tmp_path / 'ids'}") == [4, 5, 6]
