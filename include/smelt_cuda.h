@@ -353,6 +353,61 @@ SMELT_CUDA_API smelt_status smelt_cuda_dense_slots(const smelt_dense_desc* desc,
 SMELT_CUDA_API smelt_status smelt_cuda_dense_pipelines(const smelt_dense_desc* desc, const smelt_dense_layer* layers, uint32_t capacity, uint32_t max_chunk,
                                                        int prefill, char* out, size_t out_bytes, size_t* needed_bytes);
 
+/* ── stacks of mixers and feed-forwards with dense 16-bit weights (no reference counterpart) ──
+ * x <- x + N(mixer(N(x))), then x <- x + N(ff(N(x))), every N an RMS norm of its own with the weight stored around zero.
+ * Mixers: latent window attention (keys and values are projections of one cached latent, one rotated key part is shared by
+ * the heads; a layer may read an earlier layer's cache) and RWKV-style time mixing (token shift, per-channel decay, a
+ * matrix-valued state).  Feed-forwards: squared ReLU with biases, or `top` of `experts` clamped-gate experts.
+ * pad(n) below is n up to a multiple of 64, pad16 of 16, pad128 of 128, value(n) 64 / 128 / 256 / pad(n); all padding is zero.
+ * Weights image (bf16, 128-byte aligned tensors):
+ *   embedding [vocab, width], lm_head [vocab, pad(width)], every norm of the stream [pad(width)];
+ *   latent: in_proj rows query latent (q_rank, padded to pad(q_rank)) | latent (kv_rank) | key part (rot_dim) x pad(width),
+ *     the last two absent when kv_from >= 0; q_norm [pad(q_rank)], kv_norm [kv_rank]; q_proj per head pad16(dim) +
+ *     pad16(rot_dim) rows x pad(q_rank); kv_proj rows keys (heads pad16(dim)) | values (heads value(vdim)) x pad(kv_rank);
+ *     out_proj [width, heads value(vdim)]; rot_freq: rot_dims / 2 doubles, radians per position;
+ *   time mixing: in_proj rows r | k | v | g (heads dim each, padded to pad128) | decay (rank, padded to pad) x pad(width);
+ *     mu [5, pad(width)] in the order r, k, v, g, decay; w2 [heads dim, pad(rank)]; w0, bonus, head_norm [heads dim];
+ *     out_proj [width, pad(heads dim)];
+ *   dense: up [ff, pad(width)], up_bias [ff], down [width, pad(ff)], down_bias [width];
+ *   experts: router [experts, pad(width)], router_bias [experts], up [experts, 2 pad(ff), pad(width)] with gate and up rows in
+ *     turn, down [experts, width, pad(ff)].
+ * precision: the type of a prompt chunk's activations and of the latent cache; a decode step keeps activations in fp32. */
+enum { SMELT_MIXER_LATENT = 0, SMELT_MIXER_WKV = 1 };
+enum { SMELT_FF_NONE = 0, SMELT_FF_DENSE = 1, SMELT_FF_EXPERTS = 2 };
+typedef struct {
+    int32_t mixer, ff_kind;
+    int32_t heads, dim;
+    int32_t rot_dim, rot_dims, vdim, kv_rank, q_rank; /* rot_dims: rotated elements of rot_dim, in adjacent pairs */
+    int32_t kv_from;                                  /* latent: the layer whose cache this one reads; -1: its own */
+    uint32_t window;
+    float scale;
+    int32_t rank; /* time mixing: inner size of the decay */
+    int32_t ff, experts, top;
+    float limit;
+    uint64_t norm1, norm1b, norm2, norm2b;
+    uint64_t in_proj, out_proj;
+    uint64_t q_norm, kv_norm, q_proj, kv_proj, rot_freq;
+    uint64_t mu, w2, w0, bonus, head_norm;
+    uint64_t router, router_bias, up, up_bias, down, down_bias;
+} smelt_stack_layer;
+typedef struct {
+    int32_t layers, width, vocab, precision;
+    float eps, embedding_scale;
+    uint64_t embedding, lm_head, final_norm;
+} smelt_stack_desc;
+/* Decode table and prompt-chunk table, slots and pipeline names, as for the dense decoder above.  State slots, in the order of
+ * the layers: a latent ring and a ring of key parts per layer with a cache of its own; the heads' states and the previous
+ * token's mixer input per time-mixing layer.  A sequence that starts at position 0 needs nothing cleared. */
+SMELT_CUDA_API smelt_status smelt_cuda_build_stack_decoder(smelt_cuda_ctx* ctx, const smelt_stack_desc* desc, const smelt_stack_layer* layers,
+                                                           uint32_t capacity, uint32_t max_chunk, smelt_dispatch_record* records, size_t* n_records);
+SMELT_CUDA_API smelt_status smelt_cuda_build_stack_prefill_table(smelt_cuda_ctx* ctx, const smelt_stack_desc* desc, const smelt_stack_layer* layers,
+                                                                 uint32_t capacity, uint32_t max_chunk, smelt_dispatch_record* records, size_t* n_records);
+SMELT_CUDA_API smelt_status smelt_cuda_stack_cache_slots(const smelt_stack_desc* desc, const smelt_stack_layer* layers, int32_t* first_slot, int32_t* n_slots);
+SMELT_CUDA_API smelt_status smelt_cuda_stack_slots(const smelt_stack_desc* desc, const smelt_stack_layer* layers, uint32_t capacity, uint32_t max_chunk,
+                                                   int32_t* slots, uint64_t* bytes, int32_t* n_slots);
+SMELT_CUDA_API smelt_status smelt_cuda_stack_pipelines(const smelt_stack_desc* desc, const smelt_stack_layer* layers, uint32_t capacity, uint32_t max_chunk,
+                                                       int prefill, char* out, size_t out_bytes, size_t* needed_bytes);
+
 /* Typed launchers of those tables' kernels.  precision: SMELT_DENSE_BF16 or SMELT_DENSE_F32, the type T of a chunk's
  * activations and of the caches.  Weights are bf16, cols a multiple of 64 with zero padding.
  * mode: 0 y0 = fp32 product, 1 y0 += product (fp32), 2 rows below split to y0, the others through xIELU to y1, both in T

@@ -108,6 +108,24 @@ class DenseDesc(C.Structure):
                 ("final_gain", C.c_float), ("embedding", C.c_uint64), ("positions", C.c_uint64), ("loop_in", C.c_uint64), ("lm_head", C.c_uint64)]
 
 
+class StackLayer(C.Structure):
+    """``smelt_stack_layer``: one layer of a stack of mixers and feed-forwards."""
+    _fields_ = ([(n, C.c_int32) for n in ("mixer", "ff_kind", "heads", "dim", "rot_dim", "rot_dims", "vdim", "kv_rank", "q_rank", "kv_from")]
+                + [("window", C.c_uint32), ("scale", C.c_float)] + [(n, C.c_int32) for n in ("rank", "ff", "experts", "top")] + [("limit", C.c_float)]
+                + [(n, C.c_uint64) for n in ("norm1", "norm1b", "norm2", "norm2b", "in_proj", "out_proj", "q_norm", "kv_norm", "q_proj", "kv_proj", "rot_freq", "mu", "w2", "w0", "bonus",
+                                             "head_norm", "router", "router_bias", "up", "up_bias", "down", "down_bias")])
+
+
+MIXER_LATENT, MIXER_WKV = 0, 1
+FF_NONE, FF_DENSE, FF_EXPERTS = 0, 1, 2
+
+
+class StackDesc(C.Structure):
+    """``smelt_stack_desc``."""
+    _fields_ = [("layers", C.c_int32), ("width", C.c_int32), ("vocab", C.c_int32), ("precision", C.c_int32), ("eps", C.c_float), ("embedding_scale", C.c_float),
+                ("embedding", C.c_uint64), ("lm_head", C.c_uint64), ("final_norm", C.c_uint64)]
+
+
 class WindowDesc(C.Structure):
     """``smelt_window_desc``: attention over a sliding window and pooled blocks."""
     _fields_ = [("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("window", C.c_uint32), ("pool", C.c_uint32),

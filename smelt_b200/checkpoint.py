@@ -71,6 +71,11 @@ class TensorFile:
     def __init__(self, tensors: dict):
         self._t = tensors
 
+    def shape(self, name: str) -> tuple:
+        if name not in self._t:
+            raise CheckpointError(f"tensor {name} is missing")
+        return tuple(self._t[name][1].shape)
+
     def bf16(self, name: str, *shape: int) -> np.ndarray:
         if name not in self._t:
             raise CheckpointError(f"tensor {name} is missing")
@@ -100,7 +105,7 @@ def register(name: str, arch: Architecture) -> None:
 
 
 def architectures() -> list[str]:
-    from . import pesedra  # noqa: F401  (registers itself)
+    from . import kesedra, pesedra  # noqa: F401  (they register themselves)
 
     return sorted(_ARCHITECTURES)
 

@@ -33,18 +33,31 @@ __device__ __forceinline__ float xielu(float z, float rising, float falling) {
 }
 
 // Where a projection's output rows go.  Rows below `split` to y0 (row-major [M, ld0]); rows from
-// `split` on through xIELU to y1 ([M, ld1]).  split == rows when there is no second part.
+// `split` on through an activation to y1 ([M, ld1]).  split == rows when there is no second part.
 enum DenseMode : int {
-    kDenseStoreF32 = 0,  // y0 fp32
-    kDenseAddF32 = 1,    // y0 fp32, added to
-    kDenseStoreAct = 2,  // y0 and y1 in the activations' type
+    kDenseStoreF32 = 0,    // y0 fp32
+    kDenseAddF32 = 1,      // y0 fp32, added to
+    kDenseStoreAct = 2,    // y0 and y1 in the activations' type
+    kDenseStoreMixed = 3,  // y0 fp32, y1 in the activations' type
+    kDenseStoreGlu = 4,    // rows are (gate, up) pairs: y0[row / 2] = clamped_glu, in the activations' type
 };
+// Applied to the rows from `split` on; in kDenseStoreF32 kDenseDecay applies to all rows.
+enum DenseAct : int { kDenseXielu = 0, kDenseRelu2 = 1, kDenseTanh = 2, kDenseDecay = 3 };
 struct DenseOut {
     void* y0;
     void* y1;
     int ld0, ld1, split;
-    float rising, falling;
+    float rising, falling;  // xIELU; kDenseStoreGlu: rising is the clamp's limit
+    int act;
+    const bf16* bias;       // per row, added first; null: none
 };
+
+// The clamped gate of a pair: g = min(g, limit), u = clamp(u, -limit, limit), g sigmoid(1.702 g) (u + 1).
+__device__ __forceinline__ float clamped_glu(float g, float u, float limit) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
+}
 
 // y[rows] = W[rows, cols] . x, one activation row, everything but the weights in fp32 (both
 // activation types use it: a decode step keeps its activations in fp32).  cols is a multiple of
@@ -76,6 +89,13 @@ struct DenseGemmArgs {
     float* part_scratch;       // split-K partial sums and arrival counters
     size_t part_scratch_bytes;
     int* part_counters;
+    // Groups of rows with activations of their own: rows [g group_rows, ...) read X from row g x_group on (group_rows a
+    // multiple of 128; 0: one X).
+    int group_rows, x_group;
+    // Experts: `rows` are one expert's, W holds `experts` of them one behind the other; table[0].x entries follow, each
+    // {expert, first row of X and of y, rows (at most tile), 0}.  m: all rows of X.
+    const int4* table;
+    int experts, tile, max_entries;
 };
 cudaError_t launch_dense_gemm(const Launch& l, DenseType type, int mode, const DenseGemmArgs& a);
 

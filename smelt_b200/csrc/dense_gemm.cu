@@ -9,7 +9,8 @@
 // are persistent, one per SM; neighbouring units share their weight tile.  A matrix with few
 // tiles splits its columns: every part leaves fp32 sums in scratch and the last one to finish
 // adds them in split order.  Weight tiles of the first stages are requested before the wait for
-// the launch in front.
+// the launch in front.  With experts, a unit is a row tile of one expert's matrix and up to BN rows
+// of the activations that chose it, both taken from a table that an earlier launch has written.
 //
 // Every wait is bounded: on expiry the CTA raises bit 11 of the device error word, its roles stop,
 // copies and MMAs in flight are waited for (bounded too) and the tensor memory is freed.
@@ -69,7 +70,31 @@ struct GemmPlan {
     int row_tiles, token_tiles, ksplit, units;
 };
 
-template <int BN, int MODE>
+struct Unit {
+    int n0, m0, count;   // first output row, first position, positions
+    int wy, xy;          // first rows of the operands
+    int kb0, kb1, tile, part;
+};
+
+// An activation's values in place, the choice between kinds outside the loop.
+template <int N>
+__device__ __forceinline__ void activate(float (&v)[N], const DenseOut& o) {
+    switch (o.act) {
+        case kDenseRelu2:
+#pragma unroll
+            for (int j = 0; j < N; ++j) { const float z = fmaxf(v[j], 0.f); v[j] = z * z; }
+            break;
+        case kDenseTanh:
+#pragma unroll
+            for (int j = 0; j < N; ++j) v[j] = tanhf(v[j]);
+            break;
+        default:
+#pragma unroll
+            for (int j = 0; j < N; ++j) v[j] = xielu_bf16(v[j], o.rising, o.falling);
+    }
+}
+
+template <int BN, int MODE, bool EXPERTS>
 __global__ void __launch_bounds__(kGemmThreads, 1) gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x, const DenseGemmArgs a,
                                                                     const GemmPlan plan) {
     constexpr int kStages = gemm_stages(BN);
@@ -97,42 +122,61 @@ __global__ void __launch_bounds__(kGemmThreads, 1) gemm_bf16_kernel(const __grid
     const uint32_t tmem = s_tmem;
     volatile uint32_t* dead = &s_dead;
 
-    // unit -> (row tile, token tile, K range); the token tiles of a row tile are neighbours
-    auto unit_at = [&](int u, int& n0, int& m0, int& kb0, int& kb1, int& tile, int& part) {
-        part = u % plan.ksplit;
-        tile = u / plan.ksplit;
-        n0 = tile / plan.token_tiles * kBlockRows;
-        m0 = tile % plan.token_tiles * BN;
-        kb0 = (int)((long)part * kblocks / plan.ksplit);
-        kb1 = (int)((long)(part + 1) * kblocks / plan.ksplit);
+    int units = plan.units;
+    if (EXPERTS) {
+        pdl_wait();
+        units = __ldcg(&a.table[0].x) * plan.row_tiles;
+    }
+    // the token tiles of a row tile are neighbours; with experts the row tiles of a table entry are
+    auto unit_at = [&](int u) {
+        Unit t;
+        if (EXPERTS) {
+            const int4 e = __ldcg(a.table + 1 + u / plan.row_tiles);
+            t.n0 = u % plan.row_tiles * kBlockRows;
+            t.m0 = t.xy = e.y;
+            t.count = e.z;
+            t.wy = e.x * a.rows + t.n0;
+            t.kb0 = 0; t.kb1 = kblocks; t.tile = u; t.part = 0;
+        } else {
+            t.part = u % plan.ksplit;
+            t.tile = u / plan.ksplit;
+            t.n0 = t.wy = t.tile / plan.token_tiles * kBlockRows;
+            t.m0 = t.xy = t.tile % plan.token_tiles * BN;
+            if (a.group_rows) t.xy += t.n0 / a.group_rows * a.x_group;
+            t.count = min(BN, a.m - t.m0);
+            t.kb0 = (int)((long)t.part * kblocks / plan.ksplit);
+            t.kb1 = (int)((long)(t.part + 1) * kblocks / plan.ksplit);
+        }
+        return t;
     };
 
     if (warp == 0) {
         if (lane == 0) {
             uint32_t it = 0;  // stages issued so far
-            int n0, m0, kb0, kb1, tile, part;
             // the first stages' weights, ahead of the dependency
             uint32_t early = 0;
-            if ((int)blockIdx.x < plan.units) {
-                unit_at(blockIdx.x, n0, m0, kb0, kb1, tile, part);
-                for (; early < kStages && (int)early < kb1 - kb0; ++early) {
-                    mbar_arrive_expect_tx(&full[early], kStageBytes);
-                    tma_load_2d(smem + early * kStageBytes, &map_w, (kb0 + (int)early) * kBlockCols, n0, &full[early]);
+            if (!EXPERTS) {
+                if ((int)blockIdx.x < units) {
+                    const Unit t = unit_at(blockIdx.x);
+                    for (; early < kStages && (int)early < t.kb1 - t.kb0; ++early) {
+                        mbar_arrive_expect_tx(&full[early], kStageBytes);
+                        tma_load_2d(smem + early * kStageBytes, &map_w, (t.kb0 + (int)early) * kBlockCols, t.wy, &full[early]);
+                    }
                 }
+                pdl_wait();
             }
-            pdl_wait();
             bool alive = true;
-            for (int u = blockIdx.x; u < plan.units && alive; u += gridDim.x) {
-                unit_at(u, n0, m0, kb0, kb1, tile, part);
-                for (int kb = kb0; kb < kb1; ++kb, ++it) {
+            for (int u = blockIdx.x; u < units && alive; u += gridDim.x) {
+                const Unit t = unit_at(u);
+                for (int kb = t.kb0; kb < t.kb1; ++kb, ++it) {
                     const uint32_t s = it % kStages, use = it / kStages;
                     uint8_t* dst = smem + s * kStageBytes;
                     if (it >= early) {
                         if (use > 0 && !(alive = wait_alive(&empty[s], (use - 1) & 1, dead))) break;
                         mbar_arrive_expect_tx(&full[s], kStageBytes);
-                        tma_load_2d(dst, &map_w, kb * kBlockCols, n0, &full[s]);
+                        tma_load_2d(dst, &map_w, kb * kBlockCols, t.wy, &full[s]);
                     }
-                    tma_load_2d(dst + kATile, &map_x, kb * kBlockCols, m0, &full[s]);
+                    tma_load_2d(dst + kATile, &map_x, kb * kBlockCols, t.xy, &full[s]);
                 }
             }
             // no copy may land after the CTA has left
@@ -142,21 +186,20 @@ __global__ void __launch_bounds__(kGemmThreads, 1) gemm_bf16_kernel(const __grid
         if (lane == 0) {
             constexpr uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(BN >> 3) << 17) | ((uint32_t)(kBlockRows >> 4) << 24);  // f32 += bf16 x bf16, K-major both
             uint32_t it = 0, done = 0;
-            int n0, m0, kb0, kb1, tile, part;
             bool alive = true;
-            for (int u = blockIdx.x; u < plan.units && alive; u += gridDim.x, ++done) {
-                unit_at(u, n0, m0, kb0, kb1, tile, part);
+            for (int u = blockIdx.x; u < units && alive; u += gridDim.x, ++done) {
+                const Unit t = unit_at(u);
                 const uint32_t buf = done & 1, use = done >> 1;
                 if (use > 0 && !(alive = wait_alive(&acc_empty[buf], (use - 1) & 1, dead))) break;
                 tc_fence_after();
-                for (int kb = kb0; kb < kb1; ++kb, ++it) {
+                for (int kb = t.kb0; kb < t.kb1; ++kb, ++it) {
                     const uint32_t s = it % kStages;
                     if (!(alive = wait_alive(&full[s], (it / kStages) & 1, dead))) break;
                     tc_fence_after();
                     const uint32_t w = smem_u32(smem + s * kStageBytes), x = w + kATile;
 #pragma unroll
                     for (int k = 0; k < kBlockCols / 16; ++k)
-                        umma_f16(tmem + buf * BN, smem_desc_sw128(w + k * 32), smem_desc_sw128(x + k * 32), idesc, (kb != kb0 || k != 0) ? 1u : 0u);
+                        umma_f16(tmem + buf * BN, smem_desc_sw128(w + k * 32), smem_desc_sw128(x + k * 32), idesc, (kb != t.kb0 || k != 0) ? 1u : 0u);
                     umma_commit(&empty[s]);
                 }
                 if (alive) umma_commit(&acc_full[buf]);
@@ -165,13 +208,13 @@ __global__ void __launch_bounds__(kGemmThreads, 1) gemm_bf16_kernel(const __grid
             if (it > 0) mbar_poll_bounded(&empty[(it - 1) % kStages], ((it - 1) / kStages) & 1);
         }
     } else {
-        pdl_wait();
+        if (!EXPERTS) pdl_wait();
         const int quad = warp & 3, et = tid - 64;
         const uint32_t lane_base = tmem + ((uint32_t)(quad * 32) << 16);
         uint32_t done = 0;
-        int n0, m0, kb0, kb1, tile, part;
-        for (int u = blockIdx.x; u < plan.units; u += gridDim.x, ++done) {
-            unit_at(u, n0, m0, kb0, kb1, tile, part);
+        for (int u = blockIdx.x; u < units; u += gridDim.x, ++done) {
+            const Unit t = unit_at(u);
+            const int m0 = t.m0, tile = t.tile;
             const uint32_t buf = done & 1;
             bool alive = wait_alive(&acc_full[buf], (done >> 1) & 1, dead);
             if (plan.ksplit > 1) {  // the four warps meet below: they go on together or not at all
@@ -183,7 +226,7 @@ __global__ void __launch_bounds__(kGemmThreads, 1) gemm_bf16_kernel(const __grid
             }
             if (!__all_sync(0xffffffffu, alive)) break;
             tc_fence_after();
-            const int r = quad * 32 + lane, row = n0 + r, cnt = min(BN, a.m - m0);
+            const int r = quad * 32 + lane, row = t.n0 + r, cnt = t.count;
             bool finish = true;
             if (plan.ksplit > 1) {
                 float* mine = a.part_scratch + (size_t)u * (BN * kBlockRows);
@@ -223,7 +266,23 @@ __global__ void __launch_bounds__(kGemmThreads, 1) gemm_bf16_kernel(const __grid
 #pragma unroll
                         for (int j = 0; j < kChunk; ++j) v[j] = __uint_as_float(w[j / 8][j % 8]);
                     }
-                    if (row < a.rows) {
+                    if (MODE == kDenseStoreGlu) {
+                        // lanes are (gate, up) pairs: the even one takes the even positions, the odd one the odd ones
+                        const bool odd = lane & 1;
+                        bf16* y = static_cast<bf16*>(a.out.y0) + (size_t)(m0 + c0) * a.out.ld0 + row / 2;
+#pragma unroll
+                        for (int j = 0; j < kChunk; j += 2) {
+                            const float other = __shfl_xor_sync(0xffffffffu, odd ? v[j] : v[j + 1], 1);
+                            const float z = clamped_glu(odd ? other : v[j], odd ? v[j + 1] : other, a.out.rising);
+                            const int p = j + (odd ? 1 : 0);
+                            if (row < a.rows && c0 + p < cnt) y[(size_t)p * a.out.ld0] = from_f32<bf16>(z);
+                        }
+                    } else if (row < a.rows) {
+                        if (a.out.bias) {
+                            const float b = to_f32(a.out.bias[row]);
+#pragma unroll
+                            for (int j = 0; j < kChunk; ++j) v[j] += b;
+                        }
                         if (MODE == kDenseAddF32) {
                             float* y = static_cast<float*>(a.out.y0) + (size_t)(m0 + c0) * a.out.ld0 + row;
                             float old[kChunk];
@@ -232,19 +291,20 @@ __global__ void __launch_bounds__(kGemmThreads, 1) gemm_bf16_kernel(const __grid
 #pragma unroll
                             for (int j = 0; j < kChunk; ++j)
                                 if (c0 + j < cnt) y[(size_t)j * a.out.ld0] = old[j] + v[j];
-                        } else if (MODE == kDenseStoreF32) {
+                        } else if (MODE == kDenseStoreF32 || (MODE == kDenseStoreMixed && row < a.out.split)) {
                             float* y = static_cast<float*>(a.out.y0) + (size_t)(m0 + c0) * a.out.ld0 + row;
+                            if (MODE == kDenseStoreF32 && a.out.act == kDenseDecay) {
+#pragma unroll
+                                for (int j = 0; j < kChunk; ++j) v[j] = expf(-expf(v[j]));
+                            }
 #pragma unroll
                             for (int j = 0; j < kChunk; ++j)
                                 if (c0 + j < cnt) y[(size_t)j * a.out.ld0] = v[j];
                         } else {
-                            const bool act = row >= a.out.split;
+                            const bool act = MODE == kDenseStoreMixed || row >= a.out.split;
                             const int ld = act ? a.out.ld1 : a.out.ld0;
                             bf16* y = (act ? static_cast<bf16*>(a.out.y1) - a.out.split : static_cast<bf16*>(a.out.y0)) + (size_t)(m0 + c0) * ld + row;
-                            if (act) {
-#pragma unroll
-                                for (int j = 0; j < kChunk; ++j) v[j] = xielu_bf16(v[j], a.out.rising, a.out.falling);
-                            }
+                            if (act) activate(v, a.out);
 #pragma unroll
                             for (int j = 0; j < kChunk; ++j)
                                 if (c0 + j < cnt) y[(size_t)j * ld] = from_f32<bf16>(v[j]);
@@ -292,12 +352,21 @@ bool encode_rows(CUtensorMap* map, const void* base, int rows, int cols, int box
 template <int BN>
 cudaError_t launch_bf16_t(const Launch& l, int mode, const DenseGemmArgs& a, const GemmPlan& plan) {
     CUtensorMap mw, mx;
-    if (!encode_rows(&mw, a.w, a.rows, a.cols, kBlockRows) || !encode_rows(&mx, a.x, a.m, a.cols, BN)) return cudaErrorInvalidValue;
+    const int groups = a.group_rows ? (a.rows + a.group_rows - 1) / a.group_rows : 1;
+    if (!encode_rows(&mw, a.w, a.table ? a.rows * a.experts : a.rows, a.cols, kBlockRows) || !encode_rows(&mx, a.x, a.m + (groups - 1) * a.x_group, a.cols, BN)) return cudaErrorInvalidValue;
     const dim3 grid(std::min(plan.units, a.sm_count > 0 ? a.sm_count : 148)), block(kGemmThreads);
+    if (a.table) {
+        if constexpr (BN >= 32 && BN <= 128) {
+            if (mode == kDenseStoreF32) return launch_chained(l, gemm_bf16_kernel<BN, kDenseStoreF32, true>, grid, block, gemm_smem(BN), mw, mx, a, plan);
+            if (mode == kDenseStoreGlu) return launch_chained(l, gemm_bf16_kernel<BN, kDenseStoreGlu, true>, grid, block, gemm_smem(BN), mw, mx, a, plan);
+        }
+        return cudaErrorInvalidValue;
+    }
     switch (mode) {
-        case kDenseStoreF32: return launch_chained(l, gemm_bf16_kernel<BN, kDenseStoreF32>, grid, block, gemm_smem(BN), mw, mx, a, plan);
-        case kDenseAddF32: return launch_chained(l, gemm_bf16_kernel<BN, kDenseAddF32>, grid, block, gemm_smem(BN), mw, mx, a, plan);
-        case kDenseStoreAct: return launch_chained(l, gemm_bf16_kernel<BN, kDenseStoreAct>, grid, block, gemm_smem(BN), mw, mx, a, plan);
+        case kDenseStoreF32: return launch_chained(l, gemm_bf16_kernel<BN, kDenseStoreF32, false>, grid, block, gemm_smem(BN), mw, mx, a, plan);
+        case kDenseAddF32: return launch_chained(l, gemm_bf16_kernel<BN, kDenseAddF32, false>, grid, block, gemm_smem(BN), mw, mx, a, plan);
+        case kDenseStoreAct: return launch_chained(l, gemm_bf16_kernel<BN, kDenseStoreAct, false>, grid, block, gemm_smem(BN), mw, mx, a, plan);
+        case kDenseStoreMixed: return launch_chained(l, gemm_bf16_kernel<BN, kDenseStoreMixed, false>, grid, block, gemm_smem(BN), mw, mx, a, plan);
         default: return cudaErrorInvalidValue;
     }
 }
@@ -332,6 +401,11 @@ int plan_gemm(const DenseGemmArgs& a, GemmPlan* best) {
 
 cudaError_t launch_bf16(const Launch& l, int mode, const DenseGemmArgs& a) {
     GemmPlan plan;
+    if (a.table) {
+        const int row_tiles = (a.rows + kBlockRows - 1) / kBlockRows;
+        plan = GemmPlan{row_tiles, 1, 1, row_tiles * a.max_entries};
+        return a.tile == 32 ? launch_bf16_t<32>(l, mode, a, plan) : a.tile == 64 ? launch_bf16_t<64>(l, mode, a, plan) : a.tile == 128 ? launch_bf16_t<128>(l, mode, a, plan) : cudaErrorInvalidValue;
+    }
     switch (plan_gemm(a, &plan)) {
         case 16: return launch_bf16_t<16>(l, mode, a, plan);
         case 32: return launch_bf16_t<32>(l, mode, a, plan);
@@ -346,27 +420,41 @@ constexpr int kTile = 64, kStep = 32;
 
 template <int MODE>
 __device__ __forceinline__ void store_f32(const DenseOut& o, int token, int row, float v) {
+    if (o.bias) v += to_f32(o.bias[row]);
     float* y0 = static_cast<float*>(o.y0) + (size_t)token * o.ld0 + row;
-    if (MODE == kDenseAddF32) *y0 += v;
-    else if (MODE == kDenseStoreF32 || row < o.split) *y0 = v;
-    else static_cast<float*>(o.y1)[(size_t)token * o.ld1 + (row - o.split)] = xielu(v, o.rising, o.falling);
+    if (MODE == kDenseAddF32) { *y0 += v; return; }
+    if (MODE == kDenseStoreF32) { *y0 = o.act == kDenseDecay ? expf(-expf(v)) : v; return; }
+    if (row < o.split) { *y0 = v; return; }
+    const float z = fmaxf(v, 0.f);
+    static_cast<float*>(o.y1)[(size_t)token * o.ld1 + (row - o.split)] = o.act == kDenseRelu2 ? z * z : o.act == kDenseTanh ? tanhf(v) : xielu(v, o.rising, o.falling);
 }
 
-template <int MODE>
+template <int MODE, bool EXPERTS>
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const DenseGemmArgs a, DevDyn dyn) {
     __shared__ float xs[kTile][kStep + 1], ws[kTile][kStep + 1];
     pdl_trigger();
     pdl_wait();
     if (dyn_skip(dyn)) return;
     const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
-    const int n0 = blockIdx.x * kTile, m0 = blockIdx.y * kTile;
+    const int n0 = blockIdx.x * kTile;
+    int m0 = blockIdx.y * kTile, m1 = a.m;
+    const bf16* w = a.w;
     const float* x = static_cast<const float*>(a.x);
+    if (EXPERTS) {
+        if ((int)blockIdx.y >= a.table[0].x) return;
+        const int4 e = a.table[1 + blockIdx.y];
+        m0 = e.y;
+        m1 = e.y + e.z;
+        w += (size_t)e.x * a.rows * a.cols;
+    } else if (a.group_rows) {
+        x += (size_t)(n0 / a.group_rows) * a.x_group * a.cols;
+    }
     float acc[4][4] = {};
     for (int k0 = 0; k0 < a.cols; k0 += kStep) {
         for (int i = tid; i < kTile * kStep; i += 256) {
             const int r = i / kStep, c = i % kStep;
-            xs[r][c] = m0 + r < a.m ? x[(size_t)(m0 + r) * a.cols + k0 + c] : 0.f;
-            ws[r][c] = n0 + r < a.rows ? to_f32(a.w[(size_t)(n0 + r) * a.cols + k0 + c]) : 0.f;
+            xs[r][c] = m0 + r < m1 ? x[(size_t)(m0 + r) * a.cols + k0 + c] : 0.f;
+            ws[r][c] = n0 + r < a.rows ? to_f32(w[(size_t)(n0 + r) * a.cols + k0 + c]) : 0.f;
         }
         __syncthreads();
 #pragma unroll 8
@@ -384,16 +472,29 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const DenseGemmArgs a, De
 #pragma unroll
     for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
-            if (m0 + ty + 16 * i < a.m && n0 + tx + 16 * j < a.rows) store_f32<MODE>(a.out, m0 + ty + 16 * i, n0 + tx + 16 * j, acc[i][j]);
+        for (int j = 0; j < 4; ++j) {
+            const int token = m0 + ty + 16 * i, row = n0 + tx + 16 * j;
+            if (MODE == kDenseStoreGlu) {  // the row beside it is the neighbouring thread's
+                const float up = __shfl_xor_sync(0xffffffffu, acc[i][j], 1);
+                if (token < m1 && row < a.rows && (tx & 1) == 0) static_cast<float*>(a.out.y0)[(size_t)token * a.out.ld0 + row / 2] = clamped_glu(acc[i][j], up, a.out.rising);
+            } else if (token < m1 && row < a.rows) {
+                store_f32<MODE>(a.out, token, row, acc[i][j]);
+            }
+        }
 }
 
 cudaError_t launch_f32(const Launch& l, int mode, const DenseGemmArgs& a) {
-    const dim3 grid((a.rows + kTile - 1) / kTile, (a.m + kTile - 1) / kTile), block(256);
+    const dim3 grid((a.rows + kTile - 1) / kTile, a.table ? a.max_entries : (a.m + kTile - 1) / kTile), block(256);
+    if (a.table) {
+        if (a.tile != kTile) return cudaErrorInvalidValue;
+        if (mode == kDenseStoreF32) return launch_chained(l, gemm_f32_kernel<kDenseStoreF32, true>, grid, block, 0, a, dev_dyn(l));
+        if (mode == kDenseStoreGlu) return launch_chained(l, gemm_f32_kernel<kDenseStoreGlu, true>, grid, block, 0, a, dev_dyn(l));
+        return cudaErrorInvalidValue;
+    }
     switch (mode) {
-        case kDenseStoreF32: return launch_chained(l, gemm_f32_kernel<kDenseStoreF32>, grid, block, 0, a, dev_dyn(l));
-        case kDenseAddF32: return launch_chained(l, gemm_f32_kernel<kDenseAddF32>, grid, block, 0, a, dev_dyn(l));
-        case kDenseStoreAct: return launch_chained(l, gemm_f32_kernel<kDenseStoreAct>, grid, block, 0, a, dev_dyn(l));
+        case kDenseStoreF32: return launch_chained(l, gemm_f32_kernel<kDenseStoreF32, false>, grid, block, 0, a, dev_dyn(l));
+        case kDenseAddF32: return launch_chained(l, gemm_f32_kernel<kDenseAddF32, false>, grid, block, 0, a, dev_dyn(l));
+        case kDenseStoreAct: case kDenseStoreMixed: return launch_chained(l, gemm_f32_kernel<kDenseStoreAct, false>, grid, block, 0, a, dev_dyn(l));
         default: return cudaErrorInvalidValue;
     }
 }
@@ -401,7 +502,9 @@ cudaError_t launch_f32(const Launch& l, int mode, const DenseGemmArgs& a) {
 }  // namespace
 
 cudaError_t launch_dense_gemm(const Launch& l, DenseType type, int mode, const DenseGemmArgs& a) {
-    if (a.rows <= 0 || a.cols <= 0 || a.cols % 64 || a.m <= 0 || (mode != kDenseStoreAct && a.out.split != a.rows)) return cudaErrorInvalidValue;
+    if (a.rows <= 0 || a.cols <= 0 || a.cols % 64 || a.m <= 0 || (mode != kDenseStoreAct && mode != kDenseStoreMixed && a.out.split != a.rows)) return cudaErrorInvalidValue;
+    if ((a.group_rows && (a.group_rows % kBlockRows || a.x_group < a.m)) || (a.table && (a.experts <= 0 || a.max_entries <= 0 || a.group_rows)) || (mode == kDenseStoreGlu && (!a.table || a.rows % kBlockRows)))
+        return cudaErrorInvalidValue;
     if ((reinterpret_cast<uintptr_t>(a.w) | reinterpret_cast<uintptr_t>(a.x)) & 15u) return cudaErrorInvalidValue;
     return type == kDenseF32 ? launch_f32(l, mode, a) : launch_bf16(l, mode, a);
 }

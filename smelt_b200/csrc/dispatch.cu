@@ -14,6 +14,7 @@
 #include "dense.h"
 #include "glue.h"
 #include "runtime.h"
+#include "stack.h"
 
 using namespace smelt;
 
@@ -155,12 +156,40 @@ bool parse_pipeline(const char* entry, Pipeline* out) {
             {"smelt_window_attention", PK_WINDOW_ATTENTION, 0, true, true},
             {"smelt_window_decode", PK_WINDOW_DECODE, 0, true, false},
             {"argmax_f32_partials", PK_ARGMAX_F32_PARTIALS, 0, false, false},
+            // stacks of mixers and feed-forwards (stack_builder.cu)
+            {"smelt_dense_gemm_act", PK_DENSE_GEMM, kDenseStoreAct, true, true},
+            {"smelt_dense_gemm_relu2", PK_DENSE_GEMM, kDenseStoreAct, true, true},
+            {"smelt_dense_gemm_ring", PK_DENSE_GEMM, kDenseStoreAct, true, true},
+            {"smelt_dense_gemm_groups", PK_DENSE_GEMM, kDenseStoreMixed, true, true},
+            {"smelt_dense_gemm_decay", PK_DENSE_GEMM, kDenseStoreF32, true, true},
+            {"smelt_expert_gemm", PK_EXPERT_GEMM, kDenseStoreF32, true, true},
+            {"smelt_expert_gemm_glu", PK_EXPERT_GEMM, kDenseStoreGlu, true, true},
+            {"smelt_embed_rows", PK_EMBED_ROWS, 0, false, false},
+            {"smelt_matvec", PK_STACK_MATVEC, kInPlain, false, true},
+            {"smelt_matvec_norm", PK_STACK_MATVEC, kInNorm, false, true},
+            {"smelt_matvec_residual", PK_STACK_MATVEC, kInResidual, false, true},
+            {"smelt_matvec_shift", PK_STACK_MATVEC, kInShift, false, true},
+            {"smelt_matvec_experts_in", PK_STACK_MATVEC, kInExpertsIn, false, true},
+            {"smelt_matvec_experts_out", PK_STACK_MATVEC, kInExpertsOut, false, true},
+            {"smelt_residual_norm_rows", PK_RESIDUAL_NORM_ROWS, 0, true, false},
+            {"smelt_latent_append", PK_LATENT_APPEND, 0, true, true},
+            {"smelt_latent_query", PK_LATENT_QUERY, 0, true, true},
+            {"smelt_latent_scores", PK_LATENT_SCORES, 0, true, true},
+            {"smelt_latent_values", PK_LATENT_VALUES, 0, true, true},
+            {"smelt_latent_prefill", PK_LATENT_PREFILL, 0, true, true},
+            {"smelt_wkv_decode", PK_WKV_DECODE, 0, false, false},
+            {"smelt_wkv_prefill", PK_WKV_PREFILL, 0, false, false},
+            {"smelt_wkv_gate_rows", PK_WKV_GATE_ROWS, 0, true, false},
+            {"smelt_shift_mix_rows", PK_SHIFT_MIX_ROWS, 0, true, false},
+            {"smelt_moe_route", PK_MOE_ROUTE, 0, true, true},
+            {"smelt_moe_gather", PK_MOE_GATHER, 0, true, true},
+            {"smelt_moe_combine", PK_MOE_COMBINE, 0, false, true},
         };
         for (const Dense& d : dense)
             for (int t = 0; t < (d.typed ? 2 : 1); ++t)
                 if (name == (d.typed ? std::string(d.name) + (t == kDenseF32 ? "_f32" : "_bf16") : std::string(d.name))) {
                     if (d.shaped && p.cols <= 0) return false;
-                    p.kind = d.kind; p.mode = d.mode; p.bits = t; p.fixed_shape = name == "smelt_dense_matvec_xielu" || d.mode == kDenseStoreAct;
+                    p.kind = d.kind; p.mode = d.mode; p.bits = t; p.fixed_shape = starts_with(name, "smelt_dense_matvec_xielu") || starts_with(name, "smelt_dense_gemm_xielu");
                     *out = p;
                     return true;
                 }
@@ -742,17 +771,31 @@ smelt_status run_dense(Interp& in, const Pipeline& p, const Resolved& r) {
             return check_cuda(ctx, launch_dense_matvec(l, p.mode, a), p.name.c_str());
         }
         case PK_DENSE_GEMM: {
-            // name:cols:width; 0 W, 1 X [m, cols], 2 y, 3 y past the split (xielu); 5 rows, 6 m, 7 split, 8 ld of y, 9 ld past the split, 10 rising, 11 falling
+            // name:cols:width; 0 W, 1 X [m, cols], 2 y, 3 y past the split, 4 bias (optional); 5 rows, 6 m, 7 split, 8 ld of y, 9 ld past the split, 10 rising, 11 falling (xielu), 12 act
+            // _groups: the name's second number is the rows of a group, X is [groups, m, cols]; _ring: X is a ring of m rows, those filled so far are read
             NEED_BUF(0); NEED_BUF(1); NEED_BUF(2); NEED_U32(5, rows); NEED_U32(6, m); NEED_U32(7, split); NEED_U32(8, ld0);
+            if (starts_with(p.name, "smelt_dense_gemm_ring") && in.prefill && m > (uint64_t)in.start_pos + in.seq_len) m = in.start_pos + in.seq_len;
             DenseGemmArgs a = {};
             a.w = (const bf16*)r.buf[0].ptr; a.x = r.buf[1].ptr; a.rows = (int)rows; a.cols = p.cols; a.m = (int)m;
             a.out.y0 = r.buf[2].ptr; a.out.ld0 = (int)ld0; a.out.split = (int)split;
             if (split > rows || ld0 < split) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, p.name + ": split past the rows, or rows past the leading dimension");
-            NEED_BYTES(0, (size_t)rows * p.cols * 2); NEED_BYTES(1, (size_t)m * p.cols * es);
-            NEED_BYTES(2, ((size_t)(m - 1) * ld0 + split) * (p.mode == kDenseStoreAct ? es : 4));
-            if (p.fixed_shape) {
-                NEED_BUF(3); NEED_U32(9, ld1); NEED_F32(10, rising); NEED_F32(11, falling);
-                a.out.y1 = r.buf[3].ptr; a.out.ld1 = (int)ld1; a.out.rising = rising; a.out.falling = falling;
+            size_t groups = 1;
+            if (starts_with(p.name, "smelt_dense_gemm_groups")) {
+                if (p.group % 128) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, p.name + ": groups are multiples of 128 rows");
+                a.group_rows = p.group; a.x_group = (int)m;
+                groups = (rows + p.group - 1) / p.group;
+            }
+            NEED_BYTES(0, (size_t)rows * p.cols * 2); NEED_BYTES(1, groups * m * p.cols * es);
+            if (split) NEED_BYTES(2, ((size_t)(m - 1) * ld0 + split) * (p.mode == kDenseStoreAct ? es : 4));
+            if (r.buf[4].present) { NEED_BUF(4); NEED_BYTES(4, (size_t)rows * 2); a.out.bias = (const bf16*)r.buf[4].ptr; }
+            uint32_t act = starts_with(p.name, "smelt_dense_gemm_decay") ? (uint32_t)kDenseDecay : (uint32_t)kDenseXielu;
+            (void)host_u32(in, r, 12, &act);
+            a.out.act = (int)act;
+            if (p.fixed_shape) { NEED_F32(10, rising); NEED_F32(11, falling); a.out.rising = rising; a.out.falling = falling; }
+            if (p.fixed_shape || split < rows) {
+                NEED_BUF(3); NEED_U32(9, ld1);
+                a.out.y1 = r.buf[3].ptr; a.out.ld1 = (int)ld1;
+                if (ld1 < rows - split) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, p.name + ": rows past the leading dimension");
                 NEED_BYTES(3, ((size_t)(m - 1) * ld1 + (rows - split)) * es);
             }
             a.sm_count = ctx->sm_count; a.err = ctx->err_dev;
@@ -823,6 +866,257 @@ smelt_status run_dense(Interp& in, const Pipeline& p, const Resolved& r) {
 #undef NEED_F32
 }
 
+// Stacks of mixers and feed-forwards (stack_builder.cu writes these records).
+smelt_status run_stack(Interp& in, const Pipeline& p, const Resolved& r) {
+    smelt_cuda_ctx* ctx = in.ctx;
+    Launch l = make_launch(in, r);
+    const DenseType type = (DenseType)p.bits;
+    const size_t es = type == kDenseF32 ? 4 : 2;
+    auto f32 = [&](int i, float* v) { uint32_t b; const bool ok = host_u32(in, r, i, &b); if (ok) *v = as_f32(b); return ok; };
+#define NEED_F32(i, var)                                                                                  \
+    float var = 0.f;                                                                                      \
+    if (!f32(i, &var)) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, p.name + ": constant binding " #i " is missing")
+#define OPTIONAL(i, bytes, field, T)                                                                      \
+    if (r.buf[i].present) { NEED_BUF(i); NEED_BYTES(i, bytes); field = (T)r.buf[i].ptr; }
+    in.launches += 1;
+    switch (p.kind) {
+        case PK_EMBED_ROWS: {
+            // 0 table, 1 token ids, 2 x; 5 width, 6 ld, 7 rows, 9 scale
+            NEED_BUF(0); NEED_BUF(1); NEED_BUF(2); NEED_U32(5, width); NEED_U32(6, ld); NEED_U32(7, m); NEED_F32(9, scale);
+            NEED_BYTES(0, (size_t)ctx->cfg.vocab_size * width * 2); NEED_BYTES(1, (size_t)m * 4); NEED_BYTES(2, (size_t)m * ld * 4);
+            return check_cuda(ctx, launch_embed_rows(l, (const bf16*)r.buf[0].ptr, (const int32_t*)r.buf[1].ptr, (float*)r.buf[2].ptr, (int)width, (int)ld, (int)m, ctx->cfg.vocab_size, scale), p.name.c_str());
+        }
+        case PK_STACK_MATVEC: {
+            // name:cols:width; 0 W, 1 x, 2 y, 3 norm of y, 4 norm, 5 x out, 6 h out (experts_in: logits), 7 bias, 8 out, 9 before (experts: the choice), 10 mixes;
+            // 10 rows, 11 eps, 12 act (shift: rows of a group; experts: how many), 13 top, 14 limit
+            NEED_BUF(0); NEED_BUF(1); NEED_BUF(8); NEED_U32(10, rows);
+            StackMatvecArgs a = {};
+            a.w = (const bf16*)r.buf[0].ptr; a.x = (const float*)r.buf[1].ptr; a.out = (float*)r.buf[8].ptr;
+            a.rows = (int)rows; a.cols = p.cols; a.width = p.group; a.sm_count = ctx->sm_count;
+            const size_t cols = (size_t)p.cols;
+            if (p.mode == kInExpertsIn || p.mode == kInExpertsOut) {
+                NEED_BUF(9); NEED_U32(12, experts); NEED_U32(13, top);
+                if (experts == 0 || experts > 4096 || top == 0 || top > experts || top > (uint32_t)kMaxTop) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, p.name + ": bad expert counts");
+                a.experts = (int)experts; a.top = (int)top; a.chosen = (int2*)r.buf[9].ptr;
+                NEED_BYTES(0, (size_t)experts * rows * cols * 2); NEED_BYTES(9, (size_t)top * 8);
+                if (p.mode == kInExpertsIn) {
+                    NEED_BUF(6); NEED_F32(14, limit);
+                    a.limit = limit; a.logits = (const float*)r.buf[6].ptr;
+                    NEED_BYTES(6, (size_t)experts * 4); NEED_BYTES(1, cols * 4); NEED_BYTES(8, (size_t)top * rows / 2 * 4);
+                } else {
+                    NEED_BYTES(1, (size_t)top * cols * 4); NEED_BYTES(8, (size_t)rows * 4);
+                }
+                return check_cuda(ctx, launch_stack_matvec(l, p.mode, a), p.name.c_str());
+            }
+            NEED_BYTES(0, (size_t)rows * cols * 2); NEED_BYTES(1, cols * 4); NEED_BYTES(8, (size_t)rows * 4);
+            OPTIONAL(7, (size_t)rows * 2, a.bias, const bf16*);
+            if (p.mode != kInPlain) {
+                NEED_BUF(4); NEED_BYTES(4, cols * 2); NEED_F32(11, eps);
+                a.norm_w = (const bf16*)r.buf[4].ptr; a.eps = eps;
+            }
+            if (p.mode == kInResidual || p.mode == kInShift) {
+                if (r.buf[2].present) {
+                    NEED_BUF(2); NEED_BUF(3); NEED_BUF(5); NEED_BYTES(2, cols * 4); NEED_BYTES(3, cols * 2); NEED_BYTES(5, cols * 4);
+                    a.y = (const float*)r.buf[2].ptr; a.post_w = (const bf16*)r.buf[3].ptr; a.x_out = (float*)r.buf[5].ptr;
+                }
+                OPTIONAL(6, cols * 4, a.h_out, float*);
+            }
+            if (p.mode == kInShift) {
+                NEED_BUF(9); NEED_BUF(10); NEED_U32(12, group);
+                if (group == 0) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, p.name + ": empty groups");
+                a.before = (const float*)r.buf[9].ptr; a.mu = (const bf16*)r.buf[10].ptr; a.group_rows = (int)group;
+                NEED_BYTES(9, cols * 4); NEED_BYTES(10, (rows + group - 1) / group * cols * 2);
+            } else {
+                uint32_t act = kActNone;
+                (void)host_u32(in, r, 12, &act);
+                a.act = (int)act;
+            }
+            return check_cuda(ctx, launch_stack_matvec(l, p.mode, a), p.name.c_str());
+        }
+        case PK_RESIDUAL_NORM_ROWS: {
+            // 0 x, 1 y, 2 norm of y, 3 norm, 4 row list, 5 out, 6 h in fp32; 10 width, 11 ld, 12 m, 13 eps
+            NEED_BUF(0); NEED_BUF(3); NEED_BUF(5); NEED_U32(10, width); NEED_U32(11, ld); NEED_U32(12, m); NEED_F32(13, eps);
+            ResidualNormArgs a = {};
+            a.x = (float*)r.buf[0].ptr; a.norm_w = (const bf16*)r.buf[3].ptr; a.out = r.buf[5].ptr; a.width = (int)width; a.ld = (int)ld; a.m = (int)m; a.eps = eps;
+            OPTIONAL(4, (size_t)m * 4, a.rows, const int32_t*);
+            const size_t src = a.rows ? in.seq_len : m;
+            NEED_BYTES(0, src * ld * 4); NEED_BYTES(3, (size_t)ld * 2); NEED_BYTES(5, (size_t)m * ld * es);
+            OPTIONAL(1, src * ld * 4, a.y, const float*);
+            if (a.y) { NEED_BUF(2); NEED_BYTES(2, (size_t)ld * 2); a.post_w = (const bf16*)r.buf[2].ptr; }
+            OPTIONAL(6, (size_t)m * ld * 4, a.h_f32, float*);
+            return check_cuda(ctx, launch_residual_norm_rows(l, type, a), p.name.c_str());
+        }
+        case PK_WKV_DECODE: case PK_WKV_PREFILL: case PK_WKV_GATE_ROWS: case PK_SHIFT_MIX_ROWS: {
+            // 0 projections, 1 w2, 2 w0, 3 bonus, 4 norm, 5 state, 6 before, 7 h, 8 z (prefill, gate: o), 9 mixes, 10 out (gate: z; shift: mixes), 11 decays;
+            // 20 heads | dim << 16, 21 padded rank, 22 ld, 25 m, 26 eps
+            NEED_U32(20, hd); NEED_U32(21, rank); NEED_U32(22, ld); NEED_U32(25, m);
+            WkvArgs a = {};
+            a.heads = hd & 0xffff; a.dim = hd >> 16; a.rank = (int)rank; a.ld = (int)ld; a.m = (int)m; a.sm_count = ctx->sm_count;
+            const size_t width = (size_t)a.heads * a.dim, D = a.dim;
+            a.group = (int)((width + 127) / 128 * 128);
+            if (width == 0 || rank == 0 || ld == 0 || m == 0) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, p.name + ": bad geometry");
+            if (p.kind == PK_SHIFT_MIX_ROWS) {
+                NEED_BUF(6); NEED_BUF(7); NEED_BUF(9); NEED_BUF(10);
+                NEED_BYTES(6, (size_t)ld * 4); NEED_BYTES(7, (size_t)m * ld * 4); NEED_BYTES(9, (size_t)5 * ld * 2); NEED_BYTES(10, (size_t)5 * m * ld * es);
+                a.before = (float*)r.buf[6].ptr; a.h = (const float*)r.buf[7].ptr; a.mu = (const bf16*)r.buf[9].ptr; a.out = r.buf[10].ptr;
+                return check_cuda(ctx, launch_shift_mix_rows(l, type, a), p.name.c_str());
+            }
+            const bool decode = p.kind == PK_WKV_DECODE;
+            a.ldu = 4 * a.group + (decode ? a.rank : 0);
+            NEED_BUF(0); NEED_BUF(8); NEED_BYTES(0, (size_t)m * a.ldu * 4); NEED_BYTES(8, m * width * 4);
+            a.u = (const float*)r.buf[0].ptr;
+            if (p.kind == PK_WKV_GATE_ROWS) {
+                NEED_BUF(4); NEED_BUF(10); NEED_F32(26, eps);
+                a.ldz = (int)((width + 63) / 64 * 64);
+                NEED_BYTES(4, width * 2); NEED_BYTES(10, (size_t)m * a.ldz * es);
+                a.o = (const float*)r.buf[8].ptr; a.norm = (const bf16*)r.buf[4].ptr; a.out = r.buf[10].ptr; a.eps = eps;
+                return check_cuda(ctx, launch_wkv_gate_rows(l, type, a), p.name.c_str());
+            }
+            NEED_BUF(3); NEED_BUF(5); NEED_BUF(6); NEED_BUF(7);
+            NEED_BYTES(3, width * 2); NEED_BYTES(5, width * D * 4); NEED_BYTES(6, (size_t)ld * 4); NEED_BYTES(7, (size_t)m * ld * 4);
+            a.bonus = (const bf16*)r.buf[3].ptr; a.state = (float*)r.buf[5].ptr; a.before = (float*)r.buf[6].ptr; a.h = (const float*)r.buf[7].ptr; a.out = r.buf[8].ptr;
+            if (decode) {
+                NEED_BUF(1); NEED_BUF(2); NEED_BUF(4); NEED_F32(26, eps);
+                NEED_BYTES(1, width * rank * 2); NEED_BYTES(2, width * 2); NEED_BYTES(4, width * 2);
+                a.w2 = (const bf16*)r.buf[1].ptr; a.w0 = (const bf16*)r.buf[2].ptr; a.norm = (const bf16*)r.buf[4].ptr; a.eps = eps;
+                return check_cuda(ctx, launch_wkv_decode(l, a), p.name.c_str());
+            }
+            NEED_BUF(11); NEED_BYTES(11, m * width * 4);
+            a.decay = (const float*)r.buf[11].ptr;
+            return check_cuda(ctx, launch_wkv_prefill(l, a), p.name.c_str());
+        }
+        case PK_MOE_ROUTE: case PK_MOE_GATHER: case PK_MOE_COMBINE: {
+            // name:ld:width; 1 activations, 2 permuted, 3 logits, 4 choice, 5 places, 6 table, 7 rows of y, 8 y; 10 experts, 11 top, 12 m
+            NEED_BUF(4); NEED_BUF(5); NEED_U32(10, experts); NEED_U32(11, top); NEED_U32(12, m);
+            if (experts == 0 || experts > 4096 || top == 0 || top > experts || top > (uint32_t)kMaxTop || m == 0) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, p.name + ": bad expert counts");
+            MoeArgs a = {};
+            a.m = (int)m; a.experts = (int)experts; a.top = (int)top; a.width = p.group; a.ld = p.cols; a.tile = moe_tile((int)m, (int)top, (int)experts, type);
+            const size_t pairs = (size_t)m * top;
+            NEED_BYTES(4, pairs * 8); NEED_BYTES(5, pairs * 4);
+            a.chosen = (int2*)r.buf[4].ptr; a.place = (int32_t*)r.buf[5].ptr;
+            if (p.kind == PK_MOE_ROUTE) {
+                NEED_BUF(3); NEED_BUF(6); NEED_BYTES(3, (size_t)m * experts * 4);
+                NEED_BYTES(6, (1 + (size_t)moe_max_entries(a.m, a.top, a.experts, a.tile)) * 16);
+                a.logits = (const float*)r.buf[3].ptr; a.table = (int4*)r.buf[6].ptr;
+                in.launches += 1;
+                return check_cuda(ctx, launch_moe_route(l, a), p.name.c_str());
+            }
+            if (p.kind == PK_MOE_GATHER) {
+                NEED_BUF(1); NEED_BUF(2); NEED_BYTES(1, (size_t)m * a.ld * es); NEED_BYTES(2, pairs * a.ld * es);
+                a.h = r.buf[1].ptr; a.permuted = r.buf[2].ptr;
+                return check_cuda(ctx, launch_moe_gather(l, type, a), p.name.c_str());
+            }
+            NEED_BUF(7); NEED_BUF(8); NEED_BYTES(7, pairs * a.ld * 4); NEED_BYTES(8, (size_t)m * a.ld * 4);
+            a.y_rows = (const float*)r.buf[7].ptr; a.y = (float*)r.buf[8].ptr;
+            return check_cuda(ctx, launch_moe_combine(l, a), p.name.c_str());
+        }
+        case PK_EXPERT_GEMM: {
+            // name:cols:cols; 0 W [experts, rows, cols], 1 X [m top, cols], 2 y, 6 table; 5 rows, 6 m, 8 ld, 10 experts, 11 top, 13 limit (glu)
+            NEED_BUF(0); NEED_BUF(1); NEED_BUF(2); NEED_BUF(6); NEED_U32(5, rows); NEED_U32(6, m); NEED_U32(8, ld); NEED_U32(10, experts); NEED_U32(11, top);
+            if (experts == 0 || experts > 4096 || top == 0 || top > experts || top > (uint32_t)kMaxTop || m == 0) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, p.name + ": bad expert counts");
+            const bool glu = p.mode == kDenseStoreGlu;
+            const uint32_t out_cols = glu ? rows / 2 : rows;
+            if (ld < out_cols) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, p.name + ": rows past the leading dimension");
+            DenseGemmArgs a = {};
+            a.w = (const bf16*)r.buf[0].ptr; a.x = r.buf[1].ptr; a.rows = (int)rows; a.cols = p.cols; a.m = (int)(m * top);
+            a.out.y0 = r.buf[2].ptr; a.out.ld0 = (int)ld; a.out.split = (int)rows;
+            if (glu) { NEED_F32(13, limit); a.out.rising = limit; }
+            a.table = (const int4*)r.buf[6].ptr; a.experts = (int)experts; a.tile = moe_tile((int)m, (int)top, (int)experts, type);
+            a.max_entries = moe_max_entries((int)m, (int)top, (int)experts, a.tile);
+            a.sm_count = ctx->sm_count; a.err = ctx->err_dev;
+            NEED_BYTES(0, (size_t)experts * rows * p.cols * 2); NEED_BYTES(1, (size_t)a.m * p.cols * es); NEED_BYTES(2, ((size_t)(a.m - 1) * ld + out_cols) * (glu ? es : 4));
+            NEED_BYTES(6, (1 + (size_t)a.max_entries) * 16);
+            return check_cuda(ctx, launch_dense_gemm(l, type, p.mode, a), p.name.c_str());
+        }
+        default: break;
+    }
+    // latent attention, name:cols:q_rank; 0 projections, 1 q, 2 latent norm (append: 1 query norm), 3 keys and values, 4 latent ring, 5 key part ring, 6 qa (append: query latents),
+    // 7 angles, 8 sums (prefill: keys and values of the ring), 9 maxima, 10 z;
+    // 20 heads | own << 16, 21 dim | rot << 16, 22 vdim | rotated << 16, 23 rank, 24 ring, 25 m, 26 eps, 27 window, 28 scale
+    NEED_U32(20, heads); NEED_U32(21, dims); NEED_U32(22, vdims); NEED_U32(23, rank); NEED_U32(24, ring); NEED_U32(25, m);
+    LatentArgs a = {};
+    a.heads = heads & 0xffff; a.own = heads >> 16; a.dim = dims & 0xffff; a.rot = dims >> 16; a.vdim = vdims & 0xffff; a.rot_dims = vdims >> 16; a.rank = (int)rank; a.ring = ring; a.m = (int)m;
+    if (a.heads == 0 || a.dim == 0 || a.rot == 0 || a.vdim == 0 || a.rank == 0 || ring == 0 || m == 0) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, p.name + ": bad geometry");
+    a.q_rank = p.group;
+    a.dp = pad16(a.dim); a.rp = pad16(a.rot); a.vp = latent_value_pad(a.vdim); a.kr = pad64(a.rank); a.qp = pad64(a.q_rank);
+    a.q_f32 = in.prefill ? 0 : 1;
+    a.sm_count = ctx->sm_count;
+    const size_t q_rows = (size_t)a.heads * (a.dp + a.rp), qs = a.q_f32 ? 4 : es, M = m;
+    auto rings = [&]() -> smelt_status {
+        NEED_BUF(4); NEED_BUF(5); NEED_BYTES(4, (size_t)ring * a.kr * es); NEED_BYTES(5, (size_t)ring * a.rp * es);
+        a.c_ring = r.buf[4].ptr; a.rot_ring = r.buf[5].ptr;
+        return SMELT_OK;
+    };
+    auto angles = [&]() -> smelt_status {
+        NEED_BUF(7); NEED_BYTES(7, (size_t)a.rot_dims / 2 * 8);
+        a.freq = (const double*)r.buf[7].ptr;
+        return SMELT_OK;
+    };
+    auto projections = [&]() -> smelt_status {
+        NEED_BUF(0);
+        a.ldu = p.cols;
+        if (a.ldu < a.qp + (a.own ? a.rank + a.rot : 0)) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, p.name + ": projections are too short");
+        NEED_BYTES(0, M * a.ldu * 4);
+        a.u = (const float*)r.buf[0].ptr;
+        if (a.own) { NEED_BUF(2); NEED_BYTES(2, (size_t)a.rank * 2); a.kv_norm = (const bf16*)r.buf[2].ptr; }
+        return SMELT_OK;
+    };
+    auto sums = [&]() -> smelt_status {
+        a.splits = latent_splits(a, type);
+        NEED_BUF(8); NEED_BUF(9); NEED_BYTES(8, M * a.splits * a.heads * a.kr * 4); NEED_BYTES(9, M * a.splits * a.heads * 8);
+        a.part = (float*)r.buf[8].ptr; a.part_ml = (float2*)r.buf[9].ptr;
+        return SMELT_OK;
+    };
+#define STEP(f) { const smelt_status st = f(); if (st) return st; }
+    float scale = 0.f, eps = 0.f;
+    uint32_t window = 0;
+    if (f32(28, &scale)) a.scale = scale;
+    if (f32(26, &eps)) a.eps = eps;
+    if (host_u32(in, r, 27, &window)) a.window = window;
+    switch (p.kind) {
+        case PK_LATENT_APPEND:
+            STEP(rings); STEP(angles); STEP(projections);
+            NEED_BUF(1); NEED_BUF(6); NEED_BYTES(1, (size_t)a.qp * 2); NEED_BYTES(6, M * a.qp * es);
+            a.q_norm = (const bf16*)r.buf[1].ptr; a.cq = r.buf[6].ptr;
+            return check_cuda(ctx, launch_latent_append(l, type, a), p.name.c_str());
+        case PK_LATENT_QUERY: {
+            STEP(rings); STEP(angles);
+            const bool append = !in.prefill && a.own;
+            if (append) STEP(projections);
+            NEED_BUF(1); NEED_BUF(3); NEED_BUF(6); NEED_BYTES(1, M * q_rows * qs); NEED_BYTES(3, (size_t)a.heads * a.dp * a.kr * 2); NEED_BYTES(6, M * a.heads * (a.kr + a.rp) * 4);
+            a.q = r.buf[1].ptr; a.kv = (const bf16*)r.buf[3].ptr; a.qa = (float*)r.buf[6].ptr;
+            return check_cuda(ctx, launch_latent_query(l, type, a, append), p.name.c_str());
+        }
+        case PK_LATENT_SCORES:
+            STEP(rings); STEP(sums);
+            NEED_BUF(6); NEED_BYTES(6, M * a.heads * (a.kr + a.rp) * 4);
+            a.qa = (float*)r.buf[6].ptr;
+            return check_cuda(ctx, launch_latent_scores(l, type, a), p.name.c_str());
+        case PK_LATENT_VALUES:
+            STEP(sums);
+            NEED_BUF(3); NEED_BUF(10);
+            a.ldz = p.cols;
+            if (a.ldz < a.heads * a.vp) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, p.name + ": output rows are shorter than the heads");
+            NEED_BYTES(3, (size_t)a.heads * (a.dp + a.vp) * a.kr * 2); NEED_BYTES(10, M * a.ldz * qs);
+            a.kv = (const bf16*)r.buf[3].ptr; a.z = r.buf[10].ptr;
+            return check_cuda(ctx, launch_latent_values(l, type, a), p.name.c_str());
+        case PK_LATENT_PREFILL:
+            STEP(angles);
+            NEED_BUF(1); NEED_BUF(5); NEED_BUF(8); NEED_BUF(10);
+            a.ldz = p.cols;
+            if (type != kDenseBf16 || !in.prefill) return fail(ctx, SMELT_ERR_UNSUPPORTED, p.name + ": a prompt chunk in bf16");
+            if (a.ldz < a.heads * a.vp) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, p.name + ": output rows are shorter than the heads");
+            NEED_BYTES(1, M * q_rows * es); NEED_BYTES(5, (size_t)ring * a.rp * es); NEED_BYTES(8, (size_t)ring * a.heads * (a.dp + a.vp) * es); NEED_BYTES(10, M * a.ldz * es);
+            a.q = r.buf[1].ptr; a.rot_ring = r.buf[5].ptr; a.kv_rows = r.buf[8].ptr; a.z = r.buf[10].ptr;
+            return check_cuda(ctx, launch_latent_prefill(l, a), p.name.c_str());
+        default: break;
+    }
+    return fail(ctx, SMELT_ERR_UNKNOWN_PIPELINE, p.name + ": no handler");
+#undef STEP
+#undef OPTIONAL
+#undef NEED_F32
+}
+
 smelt_status run_record(Interp& in, const smelt_dispatch_record& rec_in) {
     smelt_cuda_ctx* ctx = in.ctx;
     smelt_dispatch_record rec = rec_in;
@@ -861,6 +1155,10 @@ smelt_status run_record(Interp& in, const smelt_dispatch_record& rec_in) {
         case PK_EMBED_POSITIONS: case PK_DENSE_MATVEC: case PK_DENSE_GEMM: case PK_SCALAR_NORM_ROWS: case PK_PAIR_ROWS: case PK_WINDOW_APPEND:
         case PK_WINDOW_POOL: case PK_WINDOW_ATTENTION: case PK_WINDOW_DECODE: case PK_ARGMAX_F32_PARTIALS:
             return run_dense(in, p, r);
+        case PK_EMBED_ROWS: case PK_STACK_MATVEC: case PK_RESIDUAL_NORM_ROWS: case PK_LATENT_APPEND: case PK_LATENT_QUERY: case PK_LATENT_SCORES: case PK_LATENT_VALUES:
+        case PK_LATENT_PREFILL: case PK_WKV_DECODE: case PK_WKV_PREFILL: case PK_WKV_GATE_ROWS: case PK_SHIFT_MIX_ROWS: case PK_MOE_ROUTE: case PK_MOE_GATHER: case PK_MOE_COMBINE:
+        case PK_EXPERT_GEMM:
+            return run_stack(in, p, r);
         case PK_ATTN_MLX_2PASS_2: {
             // attention.metal:1146-1153: 0 partials, 1 stats, 2 out, 3 qHeads.
             NEED_BUF(0); NEED_BUF(1); NEED_BUF(2); NEED_U32(3, nq);

@@ -91,6 +91,22 @@ enum PipeKind : int {
     PK_WINDOW_ATTENTION,
     PK_WINDOW_DECODE,
     PK_ARGMAX_F32_PARTIALS,
+    PK_EMBED_ROWS,
+    PK_STACK_MATVEC,
+    PK_RESIDUAL_NORM_ROWS,
+    PK_LATENT_APPEND,
+    PK_LATENT_QUERY,
+    PK_LATENT_SCORES,
+    PK_LATENT_VALUES,
+    PK_LATENT_PREFILL,
+    PK_WKV_DECODE,
+    PK_WKV_PREFILL,
+    PK_WKV_GATE_ROWS,
+    PK_SHIFT_MIX_ROWS,
+    PK_MOE_ROUTE,
+    PK_MOE_GATHER,
+    PK_MOE_COMBINE,
+    PK_EXPERT_GEMM,
 };
 
 struct Pipeline {

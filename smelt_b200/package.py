@@ -434,25 +434,68 @@ class Decoder:
         return out
 
 
+class DenseBuilders:
+    """The library's builder functions for one description of a decoder with dense 16-bit weights:
+    ``smelt_cuda_build_dense_*`` for a ``DenseDesc``, ``smelt_cuda_build_stack_*`` for a ``StackDesc``."""
+
+    def __init__(self, desc, layers, capacity: int, chunk: int):
+        self.desc, self.layers, self.capacity, self.chunk = desc, layers, int(capacity), int(chunk)
+        self.family = {capi.DenseDesc: "dense", capi.StackDesc: "stack"}[type(desc)]
+        self.lib = capi.load()
+
+    def table(self, prefill: bool):
+        """What writes the decode or the prompt-chunk table: (context or None, records or None, count) -> status."""
+        name = f"build_{self.family}_prefill_table" if prefill else f"build_{self.family}_decoder"
+        fn = getattr(self.lib, f"smelt_cuda_{name}")
+        return name, lambda h, t, n: fn(h, C.byref(self.desc), self.layers, self.capacity, self.chunk, t, n)
+
+    def cache_slots(self) -> list[int]:
+        first, n = C.c_int32(0), C.c_int32(0)
+        args = (C.byref(self.desc),) if self.family == "dense" else (C.byref(self.desc), self.layers)
+        st = getattr(self.lib, f"smelt_cuda_{self.family}_cache_slots")(*args, C.byref(first), C.byref(n))
+        if st != 0:
+            raise capi.SmeltError(st, "bad description")
+        return list(range(first.value, first.value + n.value))
+
+    def slots(self) -> list[tuple[int, int]]:
+        """(slot, bytes) of everything the two tables bind except the weights."""
+        fn, n = getattr(self.lib, f"smelt_cuda_{self.family}_slots"), C.c_int32(0)
+        fn(C.byref(self.desc), self.layers, self.capacity, self.chunk, None, None, C.byref(n))
+        index, size = (C.c_int32 * n.value)(), (C.c_uint64 * n.value)()
+        fn(C.byref(self.desc), self.layers, self.capacity, self.chunk, index, size, C.byref(n))
+        return list(zip(index, size))
+
+    def pipelines(self, prefill: bool) -> list[str]:
+        fn, need = getattr(self.lib, f"smelt_cuda_{self.family}_pipelines"), C.c_size_t(0)
+        fn(C.byref(self.desc), self.layers, self.capacity, self.chunk, int(prefill), None, C.c_size_t(0), C.byref(need))
+        buf = C.create_string_buffer(need.value)
+        fn(C.byref(self.desc), self.layers, self.capacity, self.chunk, int(prefill), buf, C.c_size_t(need.value), C.byref(need))
+        return [p for p in buf.value.decode().split("\n") if p]
+
+
 class DenseDecoder(Decoder):
-    """A decoder with dense 16-bit weights (``smelt_cuda_build_dense_decoder``): one sequence, fp32 logits.
+    """A decoder with dense 16-bit weights (a ``DenseDesc`` or a ``StackDesc``): one sequence, fp32 logits.
 
     A decoded token replays the captured graph; a prompt goes through the prompt-chunk table,
     ``max_chunk`` positions at a time.  precision: the type of a chunk's activations and of the
-    cache, "bfloat16" or "float32"."""
+    cache, "bfloat16" or "float32".  A sequence that starts at position 0 needs nothing cleared."""
 
     logits_dtype = np.float32
     PRECISIONS = {"bfloat16": 0, "float32": 1}
 
-    def __init__(self, ctx: capi.Context, image: np.ndarray, desc: capi.DenseDesc, layers, capacity: int, precision: str = "bfloat16", max_chunk: int = 512):
+    def __init__(self, ctx: capi.Context, image: np.ndarray, desc, layers, capacity: int, precision: str = "bfloat16", max_chunk: int = 512):
         self.ctx, self.desc, self.layers, self.capacity, self.batch, self.hybrid = ctx, desc, layers, int(capacity), 1, None
         desc.precision = self.PRECISIONS[precision]
         ctx.call("upload_weights", WEIGHTS_SLOT, image, C.c_size_t(image.nbytes))
-        lib = ctx.lib
-        chunk = self.prefill_chunk = int(min(max_chunk, capacity))
-        self.table = self._write_table(lambda h, t, n: lib.smelt_cuda_build_dense_decoder(h, C.byref(desc), layers, self.capacity, chunk, t, n), "build_dense_decoder")
-        self.n_records = len(self.table)
-        self.prefill_records = self._write_table(lambda h, t, n: lib.smelt_cuda_build_dense_prefill_table(h, C.byref(desc), layers, self.capacity, chunk, t, n), "build_dense_prefill_table")
+        self.prefill_chunk = int(min(max_chunk, capacity))
+        self.builders = DenseBuilders(desc, layers, self.capacity, self.prefill_chunk)
+        for prefill in (False, True):
+            name, fn = self.builders.table(prefill)
+            table = self._write_table(fn, name)
+            if prefill:
+                self.prefill_records = table
+            else:
+                self.table, self.n_records = table, len(table)
         self.graph_ready = False
 
     def _enqueue_chunk(self, tokens, start_pos: int, rows) -> None:
@@ -520,12 +563,11 @@ class DenseDecoder(Decoder):
         return out
 
     def cache_slots(self) -> list[int]:
-        first, n = C.c_int32(0), C.c_int32(0)
-        self.ctx._check(self.ctx.lib.smelt_cuda_dense_cache_slots(C.byref(self.desc), C.byref(first), C.byref(n)))
-        return list(range(first.value, first.value + n.value))
+        return self.builders.cache_slots()
 
     def reset_cache(self):
-        """Not needed between sequences: a row is written before a position that sees it is reached."""
+        """Not needed between sequences: a row is written before a position that sees it is reached, and a
+        recurrent state counts as zero at position 0."""
         for s in self.cache_slots():
             self.ctx.call("zero_slot", s)
 
@@ -533,7 +575,7 @@ class DenseDecoder(Decoder):
         return (capi.KvSlot * 0)()
 
     def state_slots(self):
-        return self.cache_slots()  # rings and block means: copied whole, restored only at their full length
+        return self.cache_slots()  # rings, block means and recurrent states: copied whole, restored only at their full length
 
 
 class Snapshot:
@@ -668,43 +710,34 @@ def _write_package_files(path: str, manifest: dict, image: np.ndarray, table, pr
             f.write(bytes(prefill_table))
 
 
-def write_dense_package(path: str, name: str, image: np.ndarray, desc: capi.DenseDesc, layers, entries: list, capacity: int, precision: str = "bfloat16",
+def write_dense_package(path: str, name: str, image: np.ndarray, desc, layers, entries: list, capacity: int, precision: str = "bfloat16",
                         max_chunk: int = 512) -> None:
     """Writes a decoder with dense 16-bit weights as a ``.smeltpkg`` that the package reader opens: both record
     tables, their pipelines and slots, the weights image.  entries: (tensor name, offset, size in bytes, shape)."""
-    lib = capi.load()
     os.makedirs(path, exist_ok=True)
     desc.precision = DenseDecoder.PRECISIONS[precision]
-    chunk = int(min(max_chunk, capacity))
+    builders = DenseBuilders(desc, layers, capacity, int(min(max_chunk, capacity)))
 
-    def text(prefill: int) -> list[str]:
-        need = C.c_size_t(0)
-        lib.smelt_cuda_dense_pipelines(C.byref(desc), layers, capacity, chunk, prefill, None, C.c_size_t(0), C.byref(need))
-        buf = C.create_string_buffer(need.value)
-        lib.smelt_cuda_dense_pipelines(C.byref(desc), layers, capacity, chunk, prefill, buf, C.c_size_t(need.value), C.byref(need))
-        return [p for p in buf.value.decode().split("\n") if p]
-
-    def table(build):
+    def table(prefill: bool):
+        what, build = builders.table(prefill)
         n = C.c_size_t(0)
-        st = build(None, C.byref(desc), layers, capacity, chunk, None, C.byref(n))
+        st = build(None, None, C.byref(n))
         out = (capi.DispatchRecord * n.value)()
-        st = st or build(None, C.byref(desc), layers, capacity, chunk, out, C.byref(n))
+        st = st or build(None, out, C.byref(n))
         if st != 0:
-            raise capi.SmeltError(st, "build_dense (dry run) failed")
+            raise capi.SmeltError(st, f"{what} (dry run) failed")
         return out
 
-    decode, prefill = table(lib.smelt_cuda_build_dense_decoder), table(lib.smelt_cuda_build_dense_prefill_table)
-    pipelines = text(0)
+    decode, prefill = table(False), table(True)
+    pipelines = builders.pipelines(False)
     for r in prefill:  # the dry run numbers its pipelines from 0: they follow the decode table's in the manifest
         if r.op_kind == 0:
             r.pipeline += len(pipelines)
-    pipelines += text(1)
-    n = C.c_int32(0)
-    lib.smelt_cuda_dense_slots(C.byref(desc), layers, capacity, chunk, None, None, C.byref(n))
-    index, size = (C.c_int32 * n.value)(), (C.c_uint64 * n.value)()
-    lib.smelt_cuda_dense_slots(C.byref(desc), layers, capacity, chunk, index, size, C.byref(n))
-    slots = [{"index": int(i), "name": f"windowCache_{i - KV_BASE_SLOT}" if i >= KV_BASE_SLOT else f"slot_{i}", "size_bytes": int(b), "dtype": "raw", "shape": [int(b)],
-              "category": "state" if i >= KV_BASE_SLOT else "activation"} for i, b in zip(index, size)]
+    pipelines += builders.pipelines(True)
+    state = "windowCache" if builders.family == "dense" else "mixerState"
+    kept = set(builders.cache_slots())
+    slots = [{"index": int(i), "name": f"{state}_{i - KV_BASE_SLOT}" if i in kept else f"slot_{i}", "size_bytes": int(b), "dtype": "raw", "shape": [int(b)],
+              "category": "state" if i in kept else "activation"} for i, b in builders.slots()]
     slots.append({"index": WEIGHTS_SLOT, "name": "weights", "size_bytes": 0, "dtype": "raw", "shape": [], "category": "weight"})
     manifest = {
         "version": 1, "kind": "text-generation", "architecture": "text-generation", "modelName": name,
