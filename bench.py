@@ -1,7 +1,7 @@
 #!/usr/bin/env python
 """Headline benchmark: greedy decode tokens/s of the full random-init 4-bit decoder.
 
-    python bench.py [--gpus N] [--steps K] [--warmup W] [--impl ours|reference] [--batch B] [--model affine-u4|pesedra]
+    python bench.py [--gpus N] [--steps K] [--warmup W] [--impl ours|reference] [--batch B] [--model affine-u4|pesedra|kesedra]
     python -m torch.distributed.run --nproc-per-node N ... bench.py --gpus N ...   (N > 1)
 
 A step is one decoded token of BASELINE config 4 (36 layers, hidden 4096, intermediate 12288,
@@ -428,20 +428,21 @@ def run_kernel_only(args):
 
 
 def run_dense_model(args):
-    """--model pesedra: decode and prefill of the looped dense-weight decoder at a few sizes, beside the plain
-    affine-u4 decoder at equal size, and each kernel's share of its roofline (one GPU)."""
-    from smelt_b200 import dense_bench
+    """--model pesedra / kesedra: decode and prefill of a decoder with dense 16-bit weights at a few sizes, beside its closest
+    neighbour at equal size (the plain affine-u4 decoder; Pesedra), and each kernel's share of its roofline (one GPU)."""
+    from smelt_b200 import dense_bench, stack_bench
 
     sizes = args.sizes.split(",")
     sampler = ClockSampler(0)
     sampler.start()
     sampler.mark()
-    got = dense_bench.run(sizes, args.steps, args.warmup)
+    got = (dense_bench if args.model == "pesedra" else stack_bench).run(sizes, args.steps, args.warmup)
     sampler.mark()
     peak, peak_kind = measured_peaks()
-    return {"metric": "pesedra decode tok/s (random weights)", "value": got[sizes[-1]]["pesedra"]["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": args.steps,
-            "warmup": args.warmup, "ms_per_step": got[sizes[-1]]["pesedra"]["decode_ms_per_token"], "higher_is_better": True, "dtype": "bf16 weights", "data": "synthetic",
-            "config": {"workload": "8 layer runs (5 layers, 3 of them twice), 2048-token prompt, chunks of 512", "l2_policy": "inputs larger than L2"},
+    workload = {"pesedra": "8 layer runs (5 layers, 3 of them twice)", "kesedra": "8 layers (latent attention, time mixing; dense, 4 of 16 experts)"}[args.model]
+    return {"metric": f"{args.model} decode tok/s (random weights)", "value": got[sizes[-1]][args.model]["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": args.steps,
+            "warmup": args.warmup, "ms_per_step": got[sizes[-1]][args.model]["decode_ms_per_token"], "higher_is_better": True, "dtype": "bf16 weights", "data": "synthetic",
+            "config": {"workload": workload + ", 2048-token prompt, chunks of 512", "l2_policy": "inputs larger than L2"},
             "clocks": sampler.stop(), "peak_gbs": peak, "peak_kind": peak_kind, "sizes": got}
 
 
@@ -519,13 +520,14 @@ def main():
                     help="N > 1: all-reduce + residual add as one peer-memory launch, or ncclAllReduce + elementwise_add")
     ap.add_argument("--kernel-only", action="store_true", help="time only the dominant kernel on a few synthetic weight sets (profiler captures)")
     ap.add_argument("--kernel-layers", type=int, default=6)
-    ap.add_argument("--model", default="affine-u4", choices=["affine-u4", "pesedra"], help="affine-u4: the headline workload; pesedra: the looped dense-weight decoder at --sizes beside it")
-    ap.add_argument("--sizes", default="2048,4096,5120", help="--model pesedra: widths to run (2048, 4096, 5120)")
+    ap.add_argument("--model", default="affine-u4", choices=["affine-u4", "pesedra", "kesedra"],
+                    help="affine-u4: the headline workload; pesedra, kesedra: that decoder at --sizes beside its closest neighbour")
+    ap.add_argument("--sizes", default="2048,4096,5120", help="--model pesedra / kesedra: widths to run (2048, 4096, 5120)")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3)
     if args.kernel_only:
         result = run_kernel_only(args)
-    elif args.model == "pesedra":
+    elif args.model in ("pesedra", "kesedra"):
         result = run_dense_model(args)
     else:
         result = run_reference(args) if args.impl == "reference" else run_ours(args)

@@ -424,6 +424,76 @@ SMELT_CUDA_API smelt_status smelt_cuda_embed_positions(smelt_cuda_ctx* ctx, cons
 SMELT_CUDA_API smelt_status smelt_cuda_scalar_norm_rows(smelt_cuda_ctx* ctx, int precision, const void* x_dev, const void* rows_dev, void* out_dev,
                                                         int width, int ld, int m, float gain, float eps);
 SMELT_CUDA_API smelt_status smelt_cuda_pair_rows(smelt_cuda_ctx* ctx, int precision, const void* x_dev, const void* x0_dev, void* out_dev, int ld, int m);
+/* The same product with more around it: y0 fp32 below `split` and T past it (mode 3); act: what the rows from split on go
+ * through (0 xIELU, 1 squared ReLU, 2 tanh; 3: every row of mode 0 through exp(-exp())); bias per row, first (may be null);
+ * group_rows > 0: five row groups with activations of their own, the last with the rest of the rows, X [5, m, cols]. */
+SMELT_CUDA_API smelt_status smelt_cuda_dense_gemm_ex(smelt_cuda_ctx* ctx, int precision, int mode, const void* w_dev, const void* x_dev, const void* bias_dev, void* y0_dev,
+                                                     void* y1_dev, int rows, int cols, int m, int split, int ld0, int ld1, int act, int group_rows);
+
+/* Typed launchers of the stack tables' kernels; sizes and layouts as for smelt_stack_desc, activations and caches of type T. */
+enum { SMELT_MATVEC_PLAIN = 0, SMELT_MATVEC_NORM = 1, SMELT_MATVEC_RESIDUAL = 2, SMELT_MATVEC_SHIFT = 3, SMELT_MATVEC_EXPERTS_IN = 4, SMELT_MATVEC_EXPERTS_OUT = 5 };
+typedef struct {
+    int32_t input;                 /* what the activation row is made of: SMELT_MATVEC_* */
+    int32_t rows, cols, width;     /* experts: of one expert (in: gate and up rows in turn); the norms' mean is over width */
+    int32_t group_rows;            /* shift: rows of each of the five groups but the last */
+    int32_t act;                   /* 0 none, 1 squared ReLU */
+    int32_t experts, top;
+    float eps, limit;
+    const void *w, *x, *y, *post_norm, *norm, *before, *mu, *bias, *logits; /* y, bias may be null */
+    void *x_out, *h_out, *out, *chosen;                                     /* h_out may be null; chosen: [top] {expert, weight} */
+} smelt_stack_matvec_args;
+SMELT_CUDA_API smelt_status smelt_cuda_stack_matvec(smelt_cuda_ctx* ctx, const smelt_stack_matvec_args* args, uint32_t position);
+
+SMELT_CUDA_API smelt_status smelt_cuda_embed_rows(smelt_cuda_ctx* ctx, const void* table_dev, const void* tokens_dev, void* x_dev, int width, int ld, int m, uint32_t vocab, float scale);
+/* x[r] += N(y[r]) (post_norm; y null: nothing), out[r] = N(x[r]) (norm) in T and, h_f32 not null, in fp32; rows not null: only
+ * those rows, and x stays as it is. */
+SMELT_CUDA_API smelt_status smelt_cuda_residual_norm_rows(smelt_cuda_ctx* ctx, int precision, void* x_dev, const void* y_dev, const void* post_norm_dev, const void* norm_dev,
+                                                          const void* rows_dev, void* out_dev, void* h_f32_dev, int width, int ld, int m, float eps);
+
+typedef struct {
+    int32_t heads, dim, rot_dim, rot_dims, vdim, kv_rank, q_rank;
+    int32_t own;                /* u carries a latent and a key part */
+    uint32_t window, ring;
+    float scale, eps;
+    int32_t m, ldu, ldz;
+    int32_t decode;             /* q and z fp32 whatever T is, one row */
+    const void *u, *q_norm, *kv_norm, *rot_freq, *q, *kv_proj, *kv_rows;
+    void *query_latent, *latent_ring, *rot_ring, *qa, *sums, *maxima, *z;
+} smelt_latent_args;
+/* append: u -> normed query latents and the rings.  query: q -> qa (a decode step with `own` appends as well).  scores: qa and
+ * the rings -> sums and maxima (latent_splits ranges of keys).  values: sums -> z.  prefill: q, kv_rows (kv_proj times the
+ * latent ring) and the ring of key parts -> z (bf16). */
+SMELT_CUDA_API smelt_status smelt_cuda_latent_append(smelt_cuda_ctx* ctx, int precision, const smelt_latent_args* args, uint32_t position);
+SMELT_CUDA_API smelt_status smelt_cuda_latent_query(smelt_cuda_ctx* ctx, int precision, const smelt_latent_args* args, uint32_t position);
+SMELT_CUDA_API smelt_status smelt_cuda_latent_scores(smelt_cuda_ctx* ctx, int precision, const smelt_latent_args* args, uint32_t position);
+SMELT_CUDA_API smelt_status smelt_cuda_latent_values(smelt_cuda_ctx* ctx, int precision, const smelt_latent_args* args, uint32_t position);
+SMELT_CUDA_API smelt_status smelt_cuda_latent_prefill(smelt_cuda_ctx* ctx, const smelt_latent_args* args, uint32_t position);
+SMELT_CUDA_API int smelt_cuda_latent_splits(smelt_cuda_ctx* ctx, int precision, const smelt_latent_args* args);
+
+typedef struct {
+    int32_t heads, dim, rank, ld, m;  /* rank: of the decay, padded to a multiple of 64 */
+    int32_t ldu, ldz;
+    float eps;
+    const void *u, *w2, *w0, *bonus, *norm, *decay, *h, *mu, *o;
+    void *state, *before, *out;
+} smelt_wkv_args;
+/* decode: one token from its projections to z.  shift: out = [5, m, ld] mixes.  prefill: projections and decays -> o.
+ * gate: o and the gate's projections -> z. */
+SMELT_CUDA_API smelt_status smelt_cuda_wkv_decode(smelt_cuda_ctx* ctx, const smelt_wkv_args* args, uint32_t position);
+SMELT_CUDA_API smelt_status smelt_cuda_wkv_shift(smelt_cuda_ctx* ctx, int precision, const smelt_wkv_args* args, uint32_t position);
+SMELT_CUDA_API smelt_status smelt_cuda_wkv_prefill(smelt_cuda_ctx* ctx, const smelt_wkv_args* args, uint32_t position);
+SMELT_CUDA_API smelt_status smelt_cuda_wkv_gate(smelt_cuda_ctx* ctx, int precision, const smelt_wkv_args* args);
+
+typedef struct {
+    int32_t m, experts, top, ff, width; /* up [experts, 2 pad(ff), pad(width)], down [experts, width, pad(ff)] */
+    float limit;
+    const void *logits, *h, *up, *down;                 /* logits fp32 [m, experts]; h [m, pad(width)] */
+    void *chosen, *place, *table, *permuted, *inner, *rows, *y; /* scratch: [m top] pairs, [m top] ints, 1 + experts + m top entries of 16 bytes, then T, T, fp32; y [m, pad(width)] */
+} smelt_moe_args;
+/* The experts of a prompt chunk: choice, permutation, both products, weighted sum.  stages: how many of the five launches' steps
+ * to run (1 choice and permutation, 2 gather, 3 gate and up, 4 down, 5 sum; only: that one alone, for timing). */
+SMELT_CUDA_API smelt_status smelt_cuda_moe_rows(smelt_cuda_ctx* ctx, int precision, const smelt_moe_args* args, int stages, int only);
+
 /* Attention over a window and pooled blocks.  A K (V) cache is [kv_heads, ring + blocks, row] of T, row = dim (vdim) padded
  * with zeros to 64, 128, 256 or a multiple of 64 beyond; position p lives in row p % ring, block b in row ring + b; ring must
  * be at least max(window, pool) + m - 1.  u: [m, heads dim + kv_heads (dim + vdim)] projections q | k | v, q: [m, heads, row]

@@ -132,6 +132,34 @@ class WindowDesc(C.Structure):
                 ("ring", C.c_uint32), ("blocks", C.c_uint32), ("scale", C.c_float), ("softcap", C.c_float), ("eps", C.c_float)]
 
 
+class StackMatvecArgs(C.Structure):
+    """``smelt_stack_matvec_args``."""
+    _fields_ = ([(n, C.c_int32) for n in ("input", "rows", "cols", "width", "group_rows", "act", "experts", "top")] + [("eps", C.c_float), ("limit", C.c_float)]
+                + [(n, C.c_void_p) for n in ("w", "x", "y", "post_norm", "norm", "before", "mu", "bias", "logits", "x_out", "h_out", "out", "chosen")])
+
+
+MATVEC_PLAIN, MATVEC_NORM, MATVEC_RESIDUAL, MATVEC_SHIFT, MATVEC_EXPERTS_IN, MATVEC_EXPERTS_OUT = range(6)
+
+
+class LatentArgs(C.Structure):
+    """``smelt_latent_args``."""
+    _fields_ = ([(n, C.c_int32) for n in ("heads", "dim", "rot_dim", "rot_dims", "vdim", "kv_rank", "q_rank", "own")] + [("window", C.c_uint32), ("ring", C.c_uint32), ("scale", C.c_float),
+                ("eps", C.c_float)] + [(n, C.c_int32) for n in ("m", "ldu", "ldz", "decode")]
+                + [(n, C.c_void_p) for n in ("u", "q_norm", "kv_norm", "rot_freq", "q", "kv_proj", "kv_rows", "query_latent", "latent_ring", "rot_ring", "qa", "sums", "maxima", "z")])
+
+
+class WkvArgs(C.Structure):
+    """``smelt_wkv_args``."""
+    _fields_ = ([(n, C.c_int32) for n in ("heads", "dim", "rank", "ld", "m", "ldu", "ldz")] + [("eps", C.c_float)]
+                + [(n, C.c_void_p) for n in ("u", "w2", "w0", "bonus", "norm", "decay", "h", "mu", "o", "state", "before", "out")])
+
+
+class MoeArgs(C.Structure):
+    """``smelt_moe_args``."""
+    _fields_ = ([(n, C.c_int32) for n in ("m", "experts", "top", "ff", "width")] + [("limit", C.c_float)]
+                + [(n, C.c_void_p) for n in ("logits", "h", "up", "down", "chosen", "place", "table", "permuted", "inner", "rows", "y")])
+
+
 class PackageOptions(C.Structure):
     _fields_ = [("context_capacity", C.c_uint32), ("context_limit", C.c_uint32)]
 

@@ -89,9 +89,9 @@ struct DenseGemmArgs {
     float* part_scratch;       // split-K partial sums and arrival counters
     size_t part_scratch_bytes;
     int* part_counters;
-    // Groups of rows with activations of their own: rows [g group_rows, ...) read X from row g x_group on (group_rows a
-    // multiple of 128; 0: one X).
-    int group_rows, x_group;
+    // Groups of rows with activations of their own: rows [g group_rows, (g + 1) group_rows) read X from row g x_group on, the last
+    // of the `groups` has the rest of the rows (group_rows a multiple of 128; 0: one X).
+    int group_rows, x_group, groups;
     // Experts: `rows` are one expert's, W holds `experts` of them one behind the other; table[0].x entries follow, each
     // {expert, first row of X and of y, rows (at most tile), 0}.  m: all rows of X.
     const int4* table;
@@ -156,7 +156,7 @@ inline cudaError_t launch_chained(const Launch& l, Kernel kernel, dim3 grid, dim
     attr[0].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr;
     cfg.numAttrs = l.pdl ? 1 : 0;
-    if (smem > 48 * 1024) {
+    if (smem > 16 * 1024) {  // the default limit is 48 KB together with the kernel's static shared memory
         cudaError_t e = cudaFuncSetAttribute(reinterpret_cast<const void*>(kernel), cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return e;
     }

@@ -1,6 +1,7 @@
 // Typed launchers of the dense-weight decoders' kernels.
 #include "dense.h"
 #include "runtime.h"
+#include "stack.h"
 
 using namespace smelt;
 
@@ -44,6 +45,23 @@ smelt_status smelt_cuda_dense_gemm(smelt_cuda_ctx* ctx, int precision, int mode,
     DenseGemmArgs a = {};
     a.w = (const bf16*)w; a.x = x; a.rows = rows; a.cols = cols; a.m = m;
     a.out = {y0, y1, ld0, ld1, split, rising, falling};
+    a.sm_count = ctx->sm_count; a.err = ctx->err_dev;
+    a.part_scratch = ctx->qmm_scratch; a.part_scratch_bytes = ctx->qmm_scratch_bytes; a.part_counters = ctx->qmm_counters;
+    return check_cuda(ctx, launch_dense_gemm(l, (DenseType)precision, mode, a), "dense gemm");
+}
+
+smelt_status smelt_cuda_dense_gemm_ex(smelt_cuda_ctx* ctx, int precision, int mode, const void* w, const void* x, const void* bias, void* y0, void* y1, int rows, int cols, int m,
+                                      int split, int ld0, int ld1, int act, int group_rows) {
+    Launch l;
+    smelt_status s = enter(ctx, &l);
+    if (s) return s;
+    if (!known(precision) || (mode != kDenseStoreF32 && mode != kDenseStoreAct && mode != kDenseStoreMixed) || !w || !x || (split > 0 && !y0) || (split < rows && !y1) || rows <= 0 || cols <= 0 ||
+        cols % 64 || m <= 0 || split < 0 || split > rows || act < 0 || act > 3 || group_rows < 0 || group_rows % 128 || (group_rows && rows <= (kMixes - 1) * group_rows))
+        return fail(ctx, SMELT_ERR_BAD_ARGUMENT, "dense gemm: bad arguments (cols a multiple of 64, groups of 128)");
+    DenseGemmArgs a = {};
+    a.w = (const bf16*)w; a.x = x; a.rows = rows; a.cols = cols; a.m = m;
+    a.out = {y0, y1, ld0, ld1, split, 0.f, 0.f, act, (const bf16*)bias};
+    a.group_rows = group_rows; a.x_group = group_rows ? m : 0; a.groups = group_rows ? kMixes : 0;
     a.sm_count = ctx->sm_count; a.err = ctx->err_dev;
     a.part_scratch = ctx->qmm_scratch; a.part_scratch_bytes = ctx->qmm_scratch_bytes; a.part_counters = ctx->qmm_counters;
     return check_cuda(ctx, launch_dense_gemm(l, (DenseType)precision, mode, a), "dense gemm");

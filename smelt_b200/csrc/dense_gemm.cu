@@ -142,7 +142,7 @@ __global__ void __launch_bounds__(kGemmThreads, 1) gemm_bf16_kernel(const __grid
             t.tile = u / plan.ksplit;
             t.n0 = t.wy = t.tile / plan.token_tiles * kBlockRows;
             t.m0 = t.xy = t.tile % plan.token_tiles * BN;
-            if (a.group_rows) t.xy += t.n0 / a.group_rows * a.x_group;
+            if (a.group_rows) t.xy += min(t.n0 / a.group_rows, a.groups - 1) * a.x_group;
             t.count = min(BN, a.m - t.m0);
             t.kb0 = (int)((long)t.part * kblocks / plan.ksplit);
             t.kb1 = (int)((long)(t.part + 1) * kblocks / plan.ksplit);
@@ -352,7 +352,7 @@ bool encode_rows(CUtensorMap* map, const void* base, int rows, int cols, int box
 template <int BN>
 cudaError_t launch_bf16_t(const Launch& l, int mode, const DenseGemmArgs& a, const GemmPlan& plan) {
     CUtensorMap mw, mx;
-    const int groups = a.group_rows ? (a.rows + a.group_rows - 1) / a.group_rows : 1;
+    const int groups = a.group_rows ? a.groups : 1;
     if (!encode_rows(&mw, a.w, a.table ? a.rows * a.experts : a.rows, a.cols, kBlockRows) || !encode_rows(&mx, a.x, a.m + (groups - 1) * a.x_group, a.cols, BN)) return cudaErrorInvalidValue;
     const dim3 grid(std::min(plan.units, a.sm_count > 0 ? a.sm_count : 148)), block(kGemmThreads);
     if (a.table) {
@@ -447,7 +447,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const DenseGemmArgs a, De
         m1 = e.y + e.z;
         w += (size_t)e.x * a.rows * a.cols;
     } else if (a.group_rows) {
-        x += (size_t)(n0 / a.group_rows) * a.x_group * a.cols;
+        x += (size_t)min(n0 / a.group_rows, a.groups - 1) * a.x_group * a.cols;
     }
     float acc[4][4] = {};
     for (int k0 = 0; k0 < a.cols; k0 += kStep) {
@@ -503,7 +503,7 @@ cudaError_t launch_f32(const Launch& l, int mode, const DenseGemmArgs& a) {
 
 cudaError_t launch_dense_gemm(const Launch& l, DenseType type, int mode, const DenseGemmArgs& a) {
     if (a.rows <= 0 || a.cols <= 0 || a.cols % 64 || a.m <= 0 || (mode != kDenseStoreAct && mode != kDenseStoreMixed && a.out.split != a.rows)) return cudaErrorInvalidValue;
-    if ((a.group_rows && (a.group_rows % kBlockRows || a.x_group < a.m)) || (a.table && (a.experts <= 0 || a.max_entries <= 0 || a.group_rows)) || (mode == kDenseStoreGlu && (!a.table || a.rows % kBlockRows)))
+    if ((a.group_rows && (a.group_rows % kBlockRows || a.x_group < a.m || a.groups <= 0)) || (a.table && (a.experts <= 0 || a.max_entries <= 0 || a.group_rows)) || (mode == kDenseStoreGlu && (!a.table || a.rows % kBlockRows)))
         return cudaErrorInvalidValue;
     if ((reinterpret_cast<uintptr_t>(a.w) | reinterpret_cast<uintptr_t>(a.x)) & 15u) return cudaErrorInvalidValue;
     return type == kDenseF32 ? launch_f32(l, mode, a) : launch_bf16(l, mode, a);

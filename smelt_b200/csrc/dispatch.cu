@@ -782,8 +782,9 @@ smelt_status run_dense(Interp& in, const Pipeline& p, const Resolved& r) {
             size_t groups = 1;
             if (starts_with(p.name, "smelt_dense_gemm_groups")) {
                 if (p.group % 128) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, p.name + ": groups are multiples of 128 rows");
-                a.group_rows = p.group; a.x_group = (int)m;
-                groups = (rows + p.group - 1) / p.group;
+                if (rows <= (uint32_t)(kMixes - 1) * p.group) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, p.name + ": the last group is empty");
+                a.group_rows = p.group; a.x_group = (int)m; a.groups = kMixes;
+                groups = kMixes;
             }
             NEED_BYTES(0, (size_t)rows * p.cols * 2); NEED_BYTES(1, groups * m * p.cols * es);
             if (split) NEED_BYTES(2, ((size_t)(m - 1) * ld0 + split) * (p.mode == kDenseStoreAct ? es : 4));
@@ -923,9 +924,9 @@ smelt_status run_stack(Interp& in, const Pipeline& p, const Resolved& r) {
             }
             if (p.mode == kInShift) {
                 NEED_BUF(9); NEED_BUF(10); NEED_U32(12, group);
-                if (group == 0) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, p.name + ": empty groups");
+                if (group == 0 || rows <= (kMixes - 1) * group) return fail(ctx, SMELT_ERR_BAD_ARGUMENT, p.name + ": empty groups");
                 a.before = (const float*)r.buf[9].ptr; a.mu = (const bf16*)r.buf[10].ptr; a.group_rows = (int)group;
-                NEED_BYTES(9, cols * 4); NEED_BYTES(10, (rows + group - 1) / group * cols * 2);
+                NEED_BYTES(9, cols * 4); NEED_BYTES(10, kMixes * cols * 2);
             } else {
                 uint32_t act = kActNone;
                 (void)host_u32(in, r, 12, &act);

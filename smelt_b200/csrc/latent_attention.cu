@@ -60,16 +60,28 @@ __global__ void __launch_bounds__(kThreads) latent_append_kernel(const LatentArg
     if (a.own) append_row<TC>(a, u, dyn_position(a.dyn) + (uint32_t)r, scratch[1]);
 }
 
-// qa[r][h] = [uk^T q | rotated part]; a CTA takes kThreads latent elements of one head.  The last y of
-// a decode step's grid appends instead.
+// qa[r][h] = [uk^T q | rotated part]; a CTA takes kQueryCols latent elements of one head: sixteen lanes of
+// eight elements side by side, sixteen groups of them over the rows of uk, whose first rows are
+// requested before the wait for the launch in front.  The last y of a decode step's grid appends instead.
+constexpr int kQueryCols = 128, kQueryDepth = 8;
+
 template <class TC, class TQ>
 __global__ void __launch_bounds__(kThreads) latent_query_kernel(const LatentArgs a, int append) {
     extern __shared__ float sq[];  // [dp]
     __shared__ float scratch[kWarps];
+    __shared__ __align__(16) float s_sum[16][kQueryCols + 4];
     pdl_trigger();
+    const int tid = threadIdx.x, r = blockIdx.z, h = blockIdx.y, grp = tid >> 4, c = blockIdx.x * kQueryCols + (tid & 15) * 8;
+    const bool mine = h < a.heads && c < a.kr;
+    const bf16* w = a.kv + (size_t)h * a.dp * a.kr + c;
+    uint4 buf[kQueryDepth];
+#pragma unroll
+    for (int j = 0; j < kQueryDepth; ++j) {
+        const int d = grp + 16 * j;
+        buf[j] = mine && d < a.dp ? *reinterpret_cast<const uint4*>(w + (size_t)d * a.kr) : make_uint4(0, 0, 0, 0);
+    }
     pdl_wait();
     if (dyn_skip(a.dyn)) return;
-    const int r = blockIdx.z, h = blockIdx.y;
     const uint32_t pos = dyn_position(a.dyn) + (uint32_t)r;
     if (append && h == a.heads) {
         if (blockIdx.x == 0) append_row<TC>(a, a.u, pos, scratch);
@@ -77,18 +89,33 @@ __global__ void __launch_bounds__(kThreads) latent_query_kernel(const LatentArgs
     }
     const TQ* q = static_cast<const TQ*>(a.q) + ((size_t)r * a.heads + h) * (a.dp + a.rp);
     float* qa = a.qa + ((size_t)r * a.heads + h) * (a.kr + a.rp);
-    for (int i = threadIdx.x; i < a.dp; i += kThreads) sq[i] = to_f32(q[i]);
+    for (int i = tid; i < a.dp; i += kThreads) sq[i] = to_f32(q[i]);
     if (blockIdx.x == 0)
-        for (int i = threadIdx.x; i < a.rp; i += kThreads) qa[a.kr + i] = i < a.rot ? rotated(q + a.dp, i, a.rot_dims, a.freq, pos) : 0.f;
+        for (int i = tid; i < a.rp; i += kThreads) qa[a.kr + i] = i < a.rot ? rotated(q + a.dp, i, a.rot_dims, a.freq, pos) : 0.f;
     __syncthreads();
-    const int c = blockIdx.x * kThreads + threadIdx.x;
-    if (c >= a.kr) return;
-    const bf16* w = a.kv + (size_t)h * a.dp * a.kr + c;
-    float acc[4] = {0.f, 0.f, 0.f, 0.f};
-    for (int d = 0; d < a.dp; d += 4)
+    float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    auto add = [&](const uint4& v, float x) {
+        const uint32_t p[4] = {v.x, v.y, v.z, v.w};
 #pragma unroll
-        for (int j = 0; j < 4; ++j) acc[j] = fmaf(sq[d + j], to_f32(w[(size_t)(d + j) * a.kr]), acc[j]);
-    qa[c] = (acc[0] + acc[1]) + (acc[2] + acc[3]);
+        for (int j = 0; j < 4; ++j) {
+            acc[2 * j] = fmaf(__uint_as_float(p[j] << 16), x, acc[2 * j]);
+            acc[2 * j + 1] = fmaf(__uint_as_float(p[j] & 0xFFFF0000u), x, acc[2 * j + 1]);
+        }
+    };
+#pragma unroll
+    for (int j = 0; j < kQueryDepth; ++j)
+        if (grp + 16 * j < a.dp) add(buf[j], sq[grp + 16 * j]);
+    if (mine)
+        for (int d = grp + 16 * kQueryDepth; d < a.dp; d += 16) add(*reinterpret_cast<const uint4*>(w + (size_t)d * a.kr), sq[d]);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) s_sum[grp][(tid & 15) * 8 + j] = acc[j];
+    __syncthreads();
+    if (tid < kQueryCols && blockIdx.x * kQueryCols + tid < a.kr) {
+        float v = 0.f;
+#pragma unroll
+        for (int g = 0; g < 16; ++g) v += s_sum[g][tid];
+        qa[blockIdx.x * kQueryCols + tid] = v;
+    }
 }
 
 // One CTA per (row, head), any size: tiles of one key per thread for the scores, then one latent
@@ -155,18 +182,29 @@ __global__ void __launch_bounds__(kThreads) latent_scores_simple_kernel(const La
 }
 
 // z[r][h] = uv (merged latent sum): a CTA merges the head's splits into shared memory, then its warps
-// take rows of uv, eight weights a lane.
+// take rows of uv, eight weights a lane; a warp's first rows are requested before the wait for the
+// launch in front.
+constexpr int kValueDepth = 8;  // 16-byte pieces a lane holds
+
 template <class TZ>
 __global__ void __launch_bounds__(kThreads) latent_values_kernel(const LatentArgs a, int rows_per_cta) {
-    extern __shared__ __align__(16) float sc[];  // [kr], then the splits' weights
+    extern __shared__ __align__(16) float sc[];  // [kr], then the splits' weights, then [row groups][kr] sums
     pdl_trigger();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, r = blockIdx.z, h = blockIdx.y;
-    const int v0 = blockIdx.x * rows_per_cta, v1 = min(a.vp, v0 + rows_per_cta);
+    const int v0 = blockIdx.x * rows_per_cta, v1 = min(a.vp, v0 + rows_per_cta), pieces = (a.kr + 255) / 256;  // of a row
+    const bf16* uv = a.kv + ((size_t)a.heads * a.dp + (size_t)h * a.vp) * a.kr;
+    auto load = [&](int n) {  // the warp's n-th piece: its rows are v0 + warp, v0 + warp + 8, ...
+        const int v = v0 + warp + n / pieces * kWarps, i = n % pieces * 256 + lane * 8;
+        return v < v1 && i < a.kr ? *reinterpret_cast<const uint4*>(uv + (size_t)v * a.kr + i) : make_uint4(0, 0, 0, 0);
+    };
+    uint4 buf[kValueDepth];
+#pragma unroll
+    for (int n = 0; n < kValueDepth; ++n) buf[n] = load(n);
     pdl_wait();
     if (dyn_skip(a.dyn)) return;
     // the splits' weights: exp(maximum - overall maximum) over the overall sum
     const float2* ml = a.part_ml + (size_t)r * a.splits * a.heads + h;
-    float* sw = sc + a.kr;  // [splits]
+    float* sw = sc + a.kr;
     if (warp == 0) {
         float m = -INFINITY, den = 0.f;
         for (int s = lane; s < a.splits; s += 32) {
@@ -184,31 +222,53 @@ __global__ void __launch_bounds__(kThreads) latent_values_kernel(const LatentArg
         for (int s = lane; s < a.splits; s += 32) sw[s] /= den;
     }
     __syncthreads();
-    for (int i = tid; i < a.kr; i += kThreads) {
+    // groups of threads take four latent elements each and every groups-th split
+    float* ss = sc + ((a.kr + a.splits + 3) & ~3);
+    const int cols = a.kr / 4, groups = max(1, kThreads / cols);
+    for (int x = tid; x < cols * groups; x += kThreads) {
+        const int g = x / cols, i = x % cols * 4;
         const float* p = a.part + ((size_t)r * a.splits * a.heads + h) * a.kr + i;
-        float acc = 0.f;
-#pragma unroll 4
-        for (int s = 0; s < a.splits; ++s) {
+        float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+        for (int s = g; s < a.splits; s += groups) {
             const float w = sw[s];
-            if (w != 0.f) acc = fmaf(p[(size_t)s * a.heads * a.kr], w, acc);
+            if (w != 0.f) {  // a split without keys has written no sums
+                const float4 v = *reinterpret_cast<const float4*>(p + (size_t)s * a.heads * a.kr);
+                acc.x = fmaf(v.x, w, acc.x); acc.y = fmaf(v.y, w, acc.y); acc.z = fmaf(v.z, w, acc.z); acc.w = fmaf(v.w, w, acc.w);
+            }
         }
-        sc[i] = acc;
+        *reinterpret_cast<float4*>(ss + (size_t)g * a.kr + i) = acc;
     }
     __syncthreads();
-    const bf16* uv = a.kv + ((size_t)a.heads * a.dp + (size_t)h * a.vp) * a.kr;
+    for (int i = tid; i < a.kr; i += kThreads) {
+        float v = 0.f;
+        for (int g = 0; g < groups; ++g) v += ss[(size_t)g * a.kr + i];
+        sc[i] = v;
+    }
+    __syncthreads();
     TZ* z = static_cast<TZ*>(a.z) + (size_t)r * a.ldz + (size_t)h * a.vp;
-    for (int v = v0 + warp; v < v1; v += kWarps) {
-        float acc = 0.f;
-        for (int i = lane * 8; i < a.kr; i += 256) {
-            const uint4 w = *reinterpret_cast<const uint4*>(uv + (size_t)v * a.kr + i);
-            const float4 x0 = *reinterpret_cast<const float4*>(sc + i), x1 = *reinterpret_cast<const float4*>(sc + i + 4);
-            const uint32_t q[4] = {w.x, w.y, w.z, w.w};
-            const float x[8] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
+    const int total = (v1 - v0 - warp + kWarps - 1) / kWarps * pieces;
+    float acc = 0.f;
+    for (int n0 = 0; n0 < total; n0 += kValueDepth) {
 #pragma unroll
-            for (int j = 0; j < 4; ++j) acc = fmaf(__uint_as_float(q[j] & 0xFFFF0000u), x[2 * j + 1], fmaf(__uint_as_float(q[j] << 16), x[2 * j], acc));
+        for (int j = 0; j < kValueDepth; ++j) {
+            const int n = n0 + j;
+            if (n >= total) break;
+            const int i = n % pieces * 256 + lane * 8;
+            if (i < a.kr) {
+                const float4 x0 = *reinterpret_cast<const float4*>(sc + i), x1 = *reinterpret_cast<const float4*>(sc + i + 4);
+                const uint32_t q[4] = {buf[j].x, buf[j].y, buf[j].z, buf[j].w};
+                const float x[8] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
+#pragma unroll
+                for (int k = 0; k < 4; ++k) acc = fmaf(__uint_as_float(q[k] & 0xFFFF0000u), x[2 * k + 1], fmaf(__uint_as_float(q[k] << 16), x[2 * k], acc));
+            }
+            if (n % pieces == pieces - 1) {
+                acc = warp_sum(acc);
+                if (lane == 0) z[v0 + warp + n / pieces * kWarps] = from_f32<TZ>(acc);
+                acc = 0.f;
+            }
+            buf[j] = load(n + kValueDepth);
         }
-        acc = warp_sum(acc);
-        if (lane == 0) z[v] = from_f32<TZ>(acc);
     }
 }
 
@@ -236,7 +296,7 @@ cudaError_t launch_latent_append(const Launch& l, DenseType type, LatentArgs a) 
 cudaError_t launch_latent_query(const Launch& l, DenseType type, LatentArgs a, bool append) {
     if (bad(a) || (append && (a.m != 1 || !a.u || a.ldu < a.qp + a.rank + a.rot))) return cudaErrorInvalidValue;
     a.dyn = dev_dyn(l);
-    const dim3 grid((a.kr + kThreads - 1) / kThreads, a.heads + (append ? 1 : 0), a.m), block(kThreads);
+    const dim3 grid((a.kr + kQueryCols - 1) / kQueryCols, a.heads + (append ? 1 : 0), a.m), block(kThreads);
     const size_t smem = (size_t)a.dp * sizeof(float);
     if (type == kDenseF32) return launch_chained(l, latent_query_kernel<float, float>, grid, block, smem, a, (int)append);
     return a.q_f32 ? launch_chained(l, latent_query_kernel<bf16, float>, grid, block, smem, a, (int)append) : launch_chained(l, latent_query_kernel<bf16, bf16>, grid, block, smem, a, (int)append);
@@ -258,7 +318,8 @@ cudaError_t launch_latent_values(const Launch& l, DenseType type, LatentArgs a) 
     int per = a.vp;  // rows of uv a CTA takes: enough CTAs for the GPU
     while (per > kWarps && (long)a.heads * a.m * ((a.vp + per - 1) / per) < sm) per = std::max(kWarps, per / 2);
     const dim3 grid((a.vp + per - 1) / per, a.heads, a.m), block(kThreads);
-    const size_t smem = (size_t)(a.kr + a.splits) * sizeof(float);
+    const int groups = std::max(1, kThreads / (a.kr / 4));
+    const size_t smem = (size_t)(((a.kr + a.splits + 3) & ~3) + groups * a.kr) * sizeof(float);
     return type == kDenseF32 || a.q_f32 ? launch_chained(l, latent_values_kernel<float>, grid, block, smem, a, per) : launch_chained(l, latent_values_kernel<bf16>, grid, block, smem, a, per);
 }
 

@@ -30,7 +30,7 @@ struct StackMatvecArgs {
     float* h_out;
     float eps;
     const float* before;
-    const bf16* mu;      // [groups][cols]
+    const bf16* mu;      // [kMixes][cols]
     int group_rows;      // rows of each group but the last
     const bf16* bias;    // per row, or null
     int act;
@@ -43,6 +43,7 @@ struct StackMatvecArgs {
     DevDyn dyn;
 };
 constexpr int kMaxTop = 64;
+constexpr int kMixes = 5;  // r, k, v, g, decay: groups of rows of the time mixing's input projection
 cudaError_t launch_stack_matvec(const Launch& l, int input, StackMatvecArgs a);
 
 __device__ __forceinline__ float silu(float z) { return z / (1.f + expf(-z)); }

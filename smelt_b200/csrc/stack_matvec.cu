@@ -7,6 +7,8 @@
 // the other one of two buffers.  The norm that a plain matrix follows is one factor in the
 // epilogue, its weight is applied while staging.  The weight stream (matvec.cuh) starts ahead of
 // the wait for the launch in front, except where the experts are chosen by it.
+#include <algorithm>
+
 #include "matvec.cuh"
 #include "stack.h"
 
@@ -62,10 +64,10 @@ __global__ void __launch_bounds__(kThreads, 1) stack_matvec_kernel(const StackMa
     const int tid = threadIdx.x;
     int r0 = blockIdx.x * rows_per_cta, r1 = min(IN == kInExpertsIn ? a.rows * a.top : a.rows, r0 + rows_per_cta), group = 0;
     if (IN == kInShift) {  // a CTA's rows belong to one group
-        const int per_group = (a.group_rows + rows_per_cta - 1) / rows_per_cta, groups = (a.rows + a.group_rows - 1) / a.group_rows;
-        group = min((int)blockIdx.x / per_group, groups - 1);
+        const int per_group = (a.group_rows + rows_per_cta - 1) / rows_per_cta;
+        group = min((int)blockIdx.x / per_group, kMixes - 1);
         r0 = group * a.group_rows + ((int)blockIdx.x - group * per_group) * rows_per_cta;
-        r1 = min(min(a.rows, (group + 1) * a.group_rows), r0 + rows_per_cta);
+        r1 = min(group == kMixes - 1 ? a.rows : (group + 1) * a.group_rows, r0 + rows_per_cta);
     }
     pdl_trigger();
 
@@ -202,10 +204,11 @@ cudaError_t launch_stack_matvec(const Launch& l, int input, StackMatvecArgs a) {
     if (input == kInExpertsIn) s.rows_per_cta = (s.rows_per_cta + 1) / 2 * 2;  // a pair stays in one CTA
     int grid = (rows + s.rows_per_cta - 1) / s.rows_per_cta;
     if (input == kInShift) {
-        if (a.group_rows <= 0 || !a.mu || !a.before) return cudaErrorInvalidValue;
-        const int sm = a.sm_count > 0 ? a.sm_count : 148, groups = (rows + a.group_rows - 1) / a.group_rows, last = rows - (groups - 1) * a.group_rows;
-        auto ctas = [&](int per) { return (groups - 1) * ((a.group_rows + per - 1) / per) + (last + per - 1) / per; };
-        while (ctas(s.rows_per_cta) > sm && s.rows_per_cta < a.group_rows) ++s.rows_per_cta;
+        const int last = rows - (kMixes - 1) * a.group_rows;
+        if (a.group_rows <= 0 || last <= 0 || !a.mu || !a.before) return cudaErrorInvalidValue;
+        const int sm = a.sm_count > 0 ? a.sm_count : 148;
+        auto ctas = [&](int per) { return (kMixes - 1) * ((a.group_rows + per - 1) / per) + (last + per - 1) / per; };
+        while (ctas(s.rows_per_cta) > sm && s.rows_per_cta < std::max(a.group_rows, last)) ++s.rows_per_cta;
         grid = ctas(s.rows_per_cta);
     }
     const size_t smem = s.smem() + (input == kInExpertsIn ? (size_t)a.experts * sizeof(float) : 0);

@@ -8,8 +8,9 @@
 // wkv_decode_kernel: one CTA per head, the whole step behind the projections.  The state and the
 // head's rows of W2, which do not depend on the launch in front, are requested before the wait for
 // it.  wkv_prefill_kernel: value columns are independent, so the columns of a head are cut over
-// CTAs and a column over kParts lanes that keep their keys' rows in registers for the whole chunk;
-// the chunk's operands pass through shared memory, a stage of positions at a time, two in flight.
+// CTAs, and the keys over sixteen lanes that keep their part of four columns in registers for the
+// whole chunk (packed fp32 pairs); the chunk's operands pass through shared memory, a stage of
+// positions at a time, two in flight.
 #include <algorithm>
 
 #include "stack.h"
@@ -45,6 +46,16 @@ __global__ void __launch_bounds__(kThreads) wkv_decode_kernel(const WkvArgs a, i
         for (int i = tid; i < D * D / 4; i += kThreads) cp_async16(ss + 4 * i, state + 4 * i);
         cp_async_commit();
     }
+    // W2: eight lanes a channel, 64 inner values a piece; the first pieces are held in registers
+    constexpr int kHeld = 4;
+    const int pieces = a.rank / 64, passes = (D + kThreads / 8 - 1) / (kThreads / 8), lane8 = tid & 7;
+    auto w2_piece = [&](int n) {
+        const int d = n / pieces * (kThreads / 8) + (tid >> 3);
+        return d < D ? *reinterpret_cast<const uint4*>(a.w2 + (size_t)(h * D + d) * a.rank + n % pieces * 64 + lane8 * 8) : make_uint4(0, 0, 0, 0);
+    };
+    uint4 held[kHeld];
+#pragma unroll
+    for (int n = 0; n < kHeld; ++n) held[n] = n < passes * pieces ? w2_piece(n) : make_uint4(0, 0, 0, 0);
     pdl_wait();
     if (dyn_skip(a.dyn)) {
         cp_async_wait<0>();
@@ -61,25 +72,24 @@ __global__ void __launch_bounds__(kThreads) wkv_decode_kernel(const WkvArgs a, i
     }
     for (int i = tid; i < a.rank; i += kThreads) st[i] = tanhf(u[4 * a.group + i]);
     ruk = cta_sum(ruk, s_sum[0]);  // with a barrier: st is ready
-    {
-        // eight lanes a channel
-        const int lane = tid & 7;
-        for (int d0 = 0; d0 < D; d0 += kThreads / 8) {
-            const int d = d0 + (tid >> 3);
-            float acc = 0.f;
-            if (d < D) {
-                const bf16* w = a.w2 + (size_t)(h * D + d) * a.rank;
-                for (int i = lane * 8; i < a.rank; i += 64) {
-                    const uint4 v = *reinterpret_cast<const uint4*>(w + i);
-                    const uint32_t q[4] = {v.x, v.y, v.z, v.w};
+    float inner = 0.f;
+    for (int n0 = 0; n0 < passes * pieces; n0 += kHeld) {
 #pragma unroll
-                    for (int j = 0; j < 4; ++j) acc = fmaf(__uint_as_float(q[j] & 0xFFFF0000u), st[i + 2 * j + 1], fmaf(__uint_as_float(q[j] << 16), st[i + 2 * j], acc));
-                }
-            }
-            acc += __shfl_xor_sync(0xffffffffu, acc, 4);
-            acc += __shfl_xor_sync(0xffffffffu, acc, 2);
-            acc += __shfl_xor_sync(0xffffffffu, acc, 1);
-            if (d < D && lane == 0) sw[d] = expf(-expf(acc + to_f32(a.w0[h * D + d])));
+        for (int j = 0; j < kHeld; ++j) {
+            const int n = n0 + j;
+            if (n >= passes * pieces) break;
+            const uint4 v = n0 == 0 ? held[j] : w2_piece(n);
+            const float* t = st + n % pieces * 64 + lane8 * 8;
+            const uint32_t q[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+            for (int i = 0; i < 4; ++i) inner = fmaf(__uint_as_float(q[i] & 0xFFFF0000u), t[2 * i + 1], fmaf(__uint_as_float(q[i] << 16), t[2 * i], inner));
+            if (n % pieces != pieces - 1) continue;
+            inner += __shfl_xor_sync(0xffffffffu, inner, 4);
+            inner += __shfl_xor_sync(0xffffffffu, inner, 2);
+            inner += __shfl_xor_sync(0xffffffffu, inner, 1);
+            const int d = n / pieces * (kThreads / 8) + (tid >> 3);
+            if (d < D && lane8 == 0) sw[d] = expf(-expf(inner + to_f32(a.w0[h * D + d])));
+            inner = 0.f;
         }
     }
     cp_async_wait<0>();
@@ -159,115 +169,177 @@ __global__ void __launch_bounds__(kThreads) shift_mix_rows_kernel(const WkvArgs 
 }
 
 // ── prompt chunk ────────────────────────────────────────────────────────────
-constexpr int kParts = 4;  // lanes a column
+// Two fp32 values in one register pair.
+__device__ __forceinline__ uint64_t pair2(float x, float y) {
+    uint64_t v;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(v) : "f"(x), "f"(y));
+    return v;
+}
+__device__ __forceinline__ float2 halves(uint64_t v) {
+    float2 f;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(f.x), "=f"(f.y) : "l"(v));
+    return f;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+    uint64_t d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+    uint64_t d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
 
-// KP: keys of a lane (a multiple of 4, dim <= kParts KP); COLS value columns a CTA.
-template <int KP, int COLS>
-__global__ void __launch_bounds__(COLS* kParts) wkv_prefill_kernel(const WkvArgs a) {
-    constexpr int kStage = KP > 16 ? 8 : 16;  // positions
-    constexpr int kPitch = KP + 4;  // parts of a row start in different banks
-    constexpr int kRow = kParts * kPitch, kCta = COLS * kParts;
+constexpr int kParts = 16, kLaneCols = 4, kPrefillThreads = 64, kPrefillCols = kPrefillThreads / kParts * kLaneCols, kTogether = 4;
+
+// KP keys (a multiple of 4, dim <= kParts KP) and kLaneCols value columns a lane; lane p of sixteen has the keys 64 q + 4 p + 0..3.
+// The bonus adds sum(r u k) v, its sum taken along with the others.  Four positions' sums over the
+// sixteen lanes are reduced together: sixteen values, halved with every exchange.
+template <int KP>
+__global__ void __launch_bounds__(kPrefillThreads) wkv_prefill_kernel(const WkvArgs a) {
+    constexpr int kStage = 64 / KP, kRow = kParts * KP, kQ = KP / 4;
     __shared__ __align__(16) float s_op[2][3][kStage][kRow];  // r, k, w
-    __shared__ __align__(16) float s_v[2][kStage][COLS];
-    const int D = a.dim, h = blockIdx.y, c0 = blockIdx.x * COLS, tid = threadIdx.x, part = tid % kParts, col = tid / kParts, c = c0 + col;
-    const bool live = c < D;
+    __shared__ __align__(16) float s_v[2][kStage][kPrefillCols];
+    const int D = a.dim, h = blockIdx.y, c0 = blockIdx.x * kPrefillCols, tid = threadIdx.x, part = tid % kParts, group = tid / kParts, col = c0 + group * kLaneCols;
     pdl_trigger();
     pdl_wait();
     if (dyn_skip(a.dyn)) return;
-    for (int i = tid; i < 2 * 3 * kStage * kRow; i += kCta) (&s_op[0][0][0][0])[i] = 0.f;  // keys past dim stay zero
-    for (int i = tid; i < 2 * kStage * COLS; i += kCta) (&s_v[0][0][0])[i] = 0.f;
+    for (int i = tid; i < 2 * 3 * kStage * kRow; i += kPrefillThreads) (&s_op[0][0][0][0])[i] = 0.f;  // keys past dim stay zero
+    for (int i = tid; i < 2 * kStage * kPrefillCols; i += kPrefillThreads) (&s_v[0][0][0])[i] = 0.f;
     __syncthreads();
 
     const int hd = a.heads * D;
+    const bool wide = D % 4 == 0 && a.ldu % 4 == 0 && a.group % 4 == 0;  // rows of whole 16-byte pieces
     auto issue = [&](int stage) {
         const int t0 = stage * kStage, n = min(kStage, a.m - t0), buf = stage & 1;
-        for (int i = tid; i < n * D; i += kCta) {
-            const int t = i / D, d = i % D, at = d / KP * kPitch + d % KP;
-            const float* u = a.u + (size_t)(t0 + t) * a.ldu + h * D + d;
-            cp_async4(&s_op[buf][0][t][at], u);
-            cp_async4(&s_op[buf][1][t][at], u + a.group);
-            cp_async4(&s_op[buf][2][t][at], a.decay + (size_t)(t0 + t) * hd + h * D + d);
-        }
-        for (int i = tid; i < n * COLS; i += kCta) {
-            const int t = i / COLS, j = i % COLS;
-            if (c0 + j < D) cp_async4(&s_v[buf][t][j], a.u + (size_t)(t0 + t) * a.ldu + 2 * a.group + h * D + c0 + j);
+        const float* u0 = a.u + (size_t)t0 * a.ldu + h * D;
+        const float* w0 = a.decay + (size_t)t0 * hd + h * D;
+        if (wide) {
+            const int pieces = D / 4;
+            for (int i = tid; i < n * pieces; i += kPrefillThreads) {
+                const int t = i / pieces, d = 4 * (i - t * pieces);
+                const float* u = u0 + (size_t)t * a.ldu + d;
+                cp_async16(&s_op[buf][0][t][d], u);
+                cp_async16(&s_op[buf][1][t][d], u + a.group);
+                cp_async16(&s_op[buf][2][t][d], w0 + (size_t)t * hd + d);
+            }
+            for (int i = tid; i < n * (kPrefillCols / 4); i += kPrefillThreads) {
+                const int t = i / (kPrefillCols / 4), j = i % (kPrefillCols / 4) * 4;
+                if (c0 + j < D) cp_async16(&s_v[buf][t][j], u0 + (size_t)t * a.ldu + 2 * a.group + c0 + j);
+            }
+        } else {
+            for (int i = tid; i < n * D; i += kPrefillThreads) {
+                const int t = i / D, d = i - t * D;
+                const float* u = u0 + (size_t)t * a.ldu + d;
+                cp_async4(&s_op[buf][0][t][d], u);
+                cp_async4(&s_op[buf][1][t][d], u + a.group);
+                cp_async4(&s_op[buf][2][t][d], w0 + (size_t)t * hd + d);
+            }
+            for (int i = tid; i < n * kPrefillCols; i += kPrefillThreads) {
+                const int t = i / kPrefillCols, j = i % kPrefillCols;
+                if (c0 + j < D) cp_async4(&s_v[buf][t][j], u0 + (size_t)t * a.ldu + 2 * a.group + c0 + j);
+            }
         }
         cp_async_commit();
     };
     const int stages = (a.m + kStage - 1) / kStage;
     issue(0);
 
-    float S[KP], ub[KP];
+    uint64_t S[kLaneCols][KP / 2], ub[KP / 2];
     float* state = a.state + (size_t)h * D * D;
     const bool fresh = dyn_position(a.dyn) == 0u;
 #pragma unroll
-    for (int j = 0; j < KP; ++j) {
-        const int k = part * KP + j;
-        ub[j] = k < D ? to_f32(a.bonus[h * D + k]) : 0.f;
-        S[j] = live && k < D && !fresh ? state[(size_t)k * D + c] : 0.f;
+    for (int i = 0; i < KP / 2; ++i) {
+        const int k = i / 2 * 64 + part * 4 + i % 2 * 2;
+        auto bonus = [&](int j) { return j < D ? to_f32(a.bonus[h * D + j]) : 0.f; };
+        ub[i] = pair2(bonus(k), bonus(k + 1));
+#pragma unroll
+        for (int c = 0; c < kLaneCols; ++c) {
+            auto at = [&](int j) { return j < D && col + c < D && !fresh ? state[(size_t)j * D + col + c] : 0.f; };
+            S[c][i] = pair2(at(k), at(k + 1));
+        }
     }
-    float* o = static_cast<float*>(a.out) + h * D + c;
+    float* o = static_cast<float*>(a.out) + h * D;
     for (int stage = 0; stage < stages; ++stage) {
         if (stage + 1 < stages) issue(stage + 1);
         else cp_async_commit();
         cp_async_wait<1>();
         __syncthreads();
         const int buf = stage & 1, n = min(kStage, a.m - stage * kStage);
-#pragma unroll 2
-        for (int t = 0; t < n; ++t) {
-            const float4* r4 = reinterpret_cast<const float4*>(&s_op[buf][0][t][part * kPitch]);
-            const float4* k4 = reinterpret_cast<const float4*>(&s_op[buf][1][t][part * kPitch]);
-            const float4* w4 = reinterpret_cast<const float4*>(&s_op[buf][2][t][part * kPitch]);
-            const float v = s_v[buf][t][col];
-            float acc[4] = {0.f, 0.f, 0.f, 0.f};
+        for (int t = 0; t < n; t += kTogether) {
+            float sum[kTogether * kLaneCols];
+            auto position = [&](int x) {
+                const ulonglong2* r2 = reinterpret_cast<const ulonglong2*>(&s_op[buf][0][t + x][part * 4]);
+                const ulonglong2* k2 = reinterpret_cast<const ulonglong2*>(&s_op[buf][1][t + x][part * 4]);
+                const ulonglong2* w2 = reinterpret_cast<const ulonglong2*>(&s_op[buf][2][t + x][part * 4]);
+                const float4 v4 = *reinterpret_cast<const float4*>(&s_v[buf][t + x][group * kLaneCols]);
+                const float v[kLaneCols] = {v4.x, v4.y, v4.z, v4.w};
+                uint64_t acc[kLaneCols], b = 0;
 #pragma unroll
-            for (int q = 0; q < KP / 4; ++q) {
-                const float4 r = r4[q], k = k4[q], w = w4[q];
-                const float rr[4] = {r.x, r.y, r.z, r.w}, kk[4] = {k.x, k.y, k.z, k.w}, ww[4] = {w.x, w.y, w.z, w.w};
+                for (int q = 0; q < kQ; ++q) {
+                    const ulonglong2 r = r2[q * 16], k = k2[q * 16], w = w2[q * 16];
+                    const uint64_t rr[2] = {r.x, r.y}, kk[2] = {k.x, k.y}, ww[2] = {w.x, w.y};
 #pragma unroll
-                for (int j = 0; j < 4; ++j) {
-                    const float kv = kk[j] * v;
-                    acc[j] = fmaf(rr[j], fmaf(ub[4 * q + j], kv, S[4 * q + j]), acc[j]);
-                    S[4 * q + j] = fmaf(ww[j], S[4 * q + j], kv);
+                    for (int j = 0; j < 2; ++j) {
+                        const int i = 2 * q + j;
+                        const uint64_t ru = mul2(rr[j], ub[i]);
+                        b = i == 0 ? mul2(ru, kk[j]) : fma2(ru, kk[j], b);
+#pragma unroll
+                        for (int c = 0; c < kLaneCols; ++c) {
+                            acc[c] = i == 0 ? mul2(rr[j], S[c][i]) : fma2(rr[j], S[c][i], acc[c]);
+                            S[c][i] = fma2(ww[j], S[c][i], mul2(kk[j], pair2(v[c], v[c])));
+                        }
+                    }
+                }
+                const float2 bs = halves(b);
+#pragma unroll
+                for (int c = 0; c < kLaneCols; ++c) {
+                    const float2 f = halves(acc[c]);
+                    sum[x * kLaneCols + c] = fmaf(bs.x + bs.y, v[c], f.x + f.y);
+                }
+            };
+            if (t + kTogether <= n) {
+#pragma unroll
+                for (int x = 0; x < kTogether; ++x) position(x);
+            } else {
+#pragma unroll
+                for (int x = 0; x < kTogether; ++x) {
+                    if (t + x < n) position(x);
+                    else
+#pragma unroll
+                        for (int c = 0; c < kLaneCols; ++c) sum[x * kLaneCols + c] = 0.f;
                 }
             }
-            float sum = (acc[0] + acc[1]) + (acc[2] + acc[3]);
-            sum += __shfl_xor_sync(0xffffffffu, sum, 1);
-            sum += __shfl_xor_sync(0xffffffffu, sum, 2);
-            if (part == 0 && live) o[(size_t)(stage * kStage + t) * hd] = sum;
+#pragma unroll
+            for (int off = kParts / 2; off > 0; off >>= 1) {
+                const bool up = part & off;
+#pragma unroll
+                for (int i = 0; i < off; ++i) {
+                    const float keep = up ? sum[i + off] : sum[i], send = up ? sum[i] : sum[i + off];
+                    sum[i] = keep + __shfl_xor_sync(0xffffffffu, send, off);
+                }
+            }
+            const int x = part / kLaneCols, c = col + part % kLaneCols;  // the lane's own sum
+            if (t + x < n && c < D) o[(size_t)(stage * kStage + t + x) * hd + c] = sum[0];
         }
         __syncthreads();  // the buffer may be refilled
     }
     cp_async_wait<0>();
-    if (live)
 #pragma unroll
-        for (int j = 0; j < KP; ++j)
-            if (part * KP + j < D) state[(size_t)(part * KP + j) * D + c] = S[j];
-    if (blockIdx.x == 0)
-        for (int i = h * kCta + tid; i < a.ld; i += a.heads * kCta) a.before[i] = a.h[(size_t)(a.m - 1) * a.ld + i];
-}
-
-// Any dim: one CTA per head, the state read and written in global memory, position after position.
-__global__ void __launch_bounds__(kThreads) wkv_prefill_simple_kernel(const WkvArgs a) {
-    pdl_trigger();
-    pdl_wait();
-    if (dyn_skip(a.dyn)) return;
-    const int D = a.dim, h = blockIdx.x, hd = a.heads * D;
-    const bool fresh = dyn_position(a.dyn) == 0u;
-    float* state = a.state + (size_t)h * D * D;
-    for (int c = threadIdx.x; c < D; c += kThreads)  // a thread's columns are its own
-        for (int t = 0; t < a.m; ++t) {
-            const float* u = a.u + (size_t)t * a.ldu + h * D;
-            const float v = u[2 * a.group + c];
-            float o = 0.f;
-            for (int k = 0; k < D; ++k) {
-                const float s = fresh && t == 0 ? 0.f : state[(size_t)k * D + c], kv = u[a.group + k] * v;
-                o = fmaf(u[k], fmaf(to_f32(a.bonus[h * D + k]), kv, s), o);
-                state[(size_t)k * D + c] = fmaf(a.decay[(size_t)t * hd + h * D + k], s, kv);
+    for (int i = 0; i < KP / 2; ++i) {
+        const int k = i / 2 * 64 + part * 4 + i % 2 * 2;
+#pragma unroll
+        for (int c = 0; c < kLaneCols; ++c) {
+            const float2 f = halves(S[c][i]);
+            if (col + c < D) {
+                if (k < D) state[(size_t)k * D + col + c] = f.x;
+                if (k + 1 < D) state[(size_t)(k + 1) * D + col + c] = f.y;
             }
-            static_cast<float*>(a.out)[(size_t)t * hd + h * D + c] = o;
         }
-    for (int i = h * kThreads + threadIdx.x; i < a.ld; i += a.heads * kThreads) a.before[i] = a.h[(size_t)(a.m - 1) * a.ld + i];
+    }
+    if (blockIdx.x == 0)
+        for (int i = h * kPrefillThreads + tid; i < a.ld; i += a.heads * kPrefillThreads) a.before[i] = a.h[(size_t)(a.m - 1) * a.ld + i];
 }
 
 // One warp per (row, head).
@@ -287,11 +359,52 @@ __global__ void __launch_bounds__(kThreads) wkv_gate_rows_kernel(const WkvArgs a
     for (int d = lane; d < D; d += 32) z[d] = from_f32<T>(o[d] * f * to_f32(a.norm[h * D + d]) * silu(g[d]));
 }
 
+// The same for a dim of 4 LANES: LANES lanes a head, four elements a lane, one CTA per row.
+template <class T, int LANES>
+__global__ void __launch_bounds__(kThreads) wkv_gate_vector_kernel(const WkvArgs a) {
+    pdl_trigger();
+    pdl_wait();
+    if (dyn_skip(a.dyn)) return;
+    const int r = blockIdx.x, hd = a.heads * 4 * LANES;
+    const float* o = a.o + (size_t)r * hd;
+    const float* g = a.u + (size_t)r * a.ldu + 3 * a.group;
+    T* z = static_cast<T*>(a.out) + (size_t)r * a.ldz;
+    for (int base = 0; base < hd; base += 4 * kThreads) {  // whole warps take part in the sums
+        const int i = base + 4 * threadIdx.x;
+        const bool in = i < hd;
+        const float4 v = in ? *reinterpret_cast<const float4*>(o + i) : make_float4(0.f, 0.f, 0.f, 0.f), y = in ? *reinterpret_cast<const float4*>(g + i) : v;
+        const uint2 n = in ? *reinterpret_cast<const uint2*>(a.norm + i) : make_uint2(0, 0);
+        float ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w)));
+#pragma unroll
+        for (int off = LANES / 2; off > 0; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
+        if (!in) continue;
+        const float f = rsqrtf(ss / (float)(4 * LANES) + a.eps);
+        const float4 w = make_float4(v.x * f * __uint_as_float(n.x << 16) * silu(y.x), v.y * f * __uint_as_float(n.x & 0xFFFF0000u) * silu(y.y),
+                                     v.z * f * __uint_as_float(n.y << 16) * silu(y.z), v.w * f * __uint_as_float(n.y & 0xFFFF0000u) * silu(y.w));
+        if constexpr (sizeof(T) == 4) {
+            *reinterpret_cast<float4*>(z + i) = w;
+        } else {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(w.x, w.y), hi = __floats2bfloat162_rn(w.z, w.w);
+            *reinterpret_cast<uint2*>(z + i) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+        }
+    }
+}
+
+template <class T>
+cudaError_t gate_t(const Launch& l, const WkvArgs& a) {
+    if (a.ldz % 4 == 0 && a.ldu % 4 == 0) {
+        if (a.dim == 32) return launch_chained(l, wkv_gate_vector_kernel<T, 8>, dim3(a.m), dim3(kThreads), 0, a);
+        if (a.dim == 64) return launch_chained(l, wkv_gate_vector_kernel<T, 16>, dim3(a.m), dim3(kThreads), 0, a);
+        if (a.dim == 128) return launch_chained(l, wkv_gate_vector_kernel<T, 32>, dim3(a.m), dim3(kThreads), 0, a);
+    }
+    return launch_chained(l, wkv_gate_rows_kernel<T>, dim3(a.m, (a.heads + kWarps - 1) / kWarps), dim3(kThreads), 0, a);
+}
+
 bool bad(const WkvArgs& a) { return a.heads <= 0 || a.dim <= 0 || a.group < a.heads * a.dim || a.m <= 0; }
 
-template <int KP, int COLS>
+template <int KP>
 cudaError_t prefill_t(const Launch& l, const WkvArgs& a) {
-    return launch_chained(l, wkv_prefill_kernel<KP, COLS>, dim3((a.dim + COLS - 1) / COLS, a.heads), dim3(COLS * kParts), 0, a);
+    return launch_chained(l, wkv_prefill_kernel<KP>, dim3((a.dim + kPrefillCols - 1) / kPrefillCols, a.heads), dim3(kPrefillThreads), 0, a);
 }
 
 }  // namespace
@@ -318,18 +431,15 @@ cudaError_t launch_shift_mix_rows(const Launch& l, DenseType type, WkvArgs a) {
 cudaError_t launch_wkv_prefill(const Launch& l, WkvArgs a) {
     if (bad(a)) return cudaErrorInvalidValue;
     a.dyn = dev_dyn(l);
-    if (a.dim <= 16) return prefill_t<4, 16>(l, a);
-    if (a.dim <= 32) return prefill_t<8, 16>(l, a);
-    if (a.dim <= 64) return prefill_t<16, 16>(l, a);
-    if (a.dim <= 128) return prefill_t<32, 16>(l, a);
-    return launch_chained(l, wkv_prefill_simple_kernel, dim3(a.heads), dim3(kThreads), 0, a);
+    if (a.dim <= 64) return prefill_t<4>(l, a);
+    if (a.dim <= 128) return prefill_t<8>(l, a);
+    return a.dim <= 256 ? prefill_t<16>(l, a) : cudaErrorInvalidValue;
 }
 
 cudaError_t launch_wkv_gate_rows(const Launch& l, DenseType type, WkvArgs a) {
     if (bad(a) || a.ldz < a.heads * a.dim) return cudaErrorInvalidValue;
     a.dyn = dev_dyn(l);
-    const dim3 grid(a.m, (a.heads + kWarps - 1) / kWarps), block(kThreads);
-    return type == kDenseF32 ? launch_chained(l, wkv_gate_rows_kernel<float>, grid, block, 0, a) : launch_chained(l, wkv_gate_rows_kernel<bf16>, grid, block, 0, a);
+    return type == kDenseF32 ? gate_t<float>(l, a) : gate_t<bf16>(l, a);
 }
 
 }  // namespace smelt
