@@ -1,13 +1,19 @@
 """Decode and prefill throughput of a stack of latent attention, time mixing and expert layers (Kesedra)
 beside the looped dense-weight decoder (Pesedra) at equal sizes, and both designs' kernels against their rooflines.
 
+    python -m smelt_b200.stack_bench --size 4096 --only "time mixing recurrence" [--alone] [--reps 10]
+
+times the kernels of the steps whose name contains --only (profiler captures); ``bench.py --model kesedra`` runs all.
+
 Random weights.  Sizes are width / feed-forward / heads; eight layers of each design (Kesedra: latent attention +
 dense, latent attention on the same cache + experts, time mixing + dense, time mixing + experts, twice).  Kernels are
 timed as ``kernel_bench`` times everything: a recorded pass over operand sets larger than L2, replayed between events.
 """
 from __future__ import annotations
 
+import argparse
 import ctypes as C
+import json
 
 import numpy as np
 
@@ -258,9 +264,10 @@ class Bench(kernel_bench.Bench):
             b.free()
 
 
-def kernels(size, reps=10, only=""):
+def kernels(size, reps=10, only="", alone=False):
     """Each kernel beside Pesedra's (or the DeltaNet mixer's) like kernel: share of the roofline (the larger of bytes over
-    the measured copy bandwidth and operations over the measured bf16 rate, over the time)."""
+    the measured copy bandwidth and operations over the measured bf16 rate, over the time).  only: the steps whose name
+    contains it; alone: without the like kernels."""
     width = int(size)
     ff, heads, q_rank, rank, expert_ff = SIZES[size]
     b, peak = Bench(reps, quiet=True), dense_bench.peak_tflops()
@@ -314,7 +321,7 @@ def kernels(size, reps=10, only=""):
         if only and only not in name:
             continue
         a = share(ours)
-        if like is None:
+        if like is None or alone:
             out.append({"step": name, "kesedra": a})
             continue
         c = share(like)
@@ -326,3 +333,18 @@ def kernels(size, reps=10, only=""):
 def run(sizes, steps, warmup, prompt_len=2048):
     return {size: {"size": {"width": int(size), **dict(zip(("ff", "heads", "q_rank", "decay_rank", "expert_ff"), SIZES[size]))}, "kernels": kernels(size),
                    **models(size, steps, warmup, prompt_len)} for size in sizes}
+
+
+def main():
+    ap = argparse.ArgumentParser(prog="smelt_b200.stack_bench")
+    ap.add_argument("--size", default="4096", choices=list(SIZES))
+    ap.add_argument("--only", default="")
+    ap.add_argument("--reps", type=int, default=10)
+    ap.add_argument("--alone", action="store_true", help="without the like kernels")
+    args = ap.parse_args()
+    for row in kernels(args.size, args.reps, args.only, args.alone):
+        print(json.dumps(row), flush=True)
+
+
+if __name__ == "__main__":
+    main()

@@ -125,4 +125,4 @@ def close_calls(cfg: dict, t: dict, m, toks, margin: float) -> float:
         m.feed(toks)
     finally:
         ref.route = kept
-    return float(np.mean(np.concatenate(gaps) < margin))
+    return float(np.mean(np.concatenate(gaps) < margin)) if gaps else 0.0
