@@ -49,7 +49,7 @@ struct DenseOut {
     int ld0, ld1, split;
     float rising, falling;  // xIELU; kDenseStoreGlu: rising is the clamp's limit
     int act;
-    const bf16* bias;       // per row, added first; null: none
+    const bf16* bias;       // per row, added first; null: none (kDenseAddF32 takes none)
 };
 
 // The clamped gate of a pair: g = min(g, limit), u = clamp(u, -limit, limit), g sigmoid(1.702 g) (u + 1).

@@ -76,25 +76,19 @@ struct Unit {
     int kb0, kb1, tile, part;
 };
 
-// An activation's values in place, the choice between kinds outside the loop.
-template <int N>
+template <int ACT, int N>
 __device__ __forceinline__ void activate(float (&v)[N], const DenseOut& o) {
-    switch (o.act) {
-        case kDenseRelu2:
 #pragma unroll
-            for (int j = 0; j < N; ++j) { const float z = fmaxf(v[j], 0.f); v[j] = z * z; }
-            break;
-        case kDenseTanh:
-#pragma unroll
-            for (int j = 0; j < N; ++j) v[j] = tanhf(v[j]);
-            break;
-        default:
-#pragma unroll
-            for (int j = 0; j < N; ++j) v[j] = xielu_bf16(v[j], o.rising, o.falling);
+    for (int j = 0; j < N; ++j) {
+        if (ACT == kDenseRelu2) { const float z = fmaxf(v[j], 0.f); v[j] = z * z; }
+        else if (ACT == kDenseTanh) v[j] = tanhf(v[j]);
+        else if (ACT == kDenseDecay) v[j] = expf(-expf(v[j]));
+        else v[j] = xielu_bf16(v[j], o.rising, o.falling);
     }
 }
 
-template <int BN, int MODE, bool EXPERTS>
+// ACT: what the rows past the split go through; kDenseStoreF32: kDenseDecay, or anything else for nothing.
+template <int BN, int MODE, int ACT, bool EXPERTS>
 __global__ void __launch_bounds__(kGemmThreads, 1) gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x, const DenseGemmArgs a,
                                                                     const GemmPlan plan) {
     constexpr int kStages = gemm_stages(BN);
@@ -252,6 +246,13 @@ __global__ void __launch_bounds__(kGemmThreads, 1) gemm_bf16_kernel(const __grid
                 const float* parts = a.part_scratch + (size_t)tile * plan.ksplit * (BN * kBlockRows) + r;
                 for (int c0 = 0; c0 < cnt; c0 += kChunk) {  // positions, kChunk at a time: their loads are in flight together
                     float v[kChunk];
+                    float old[MODE == kDenseAddF32 ? kChunk : 1];
+                    if (MODE == kDenseAddF32 && row < a.rows) {  // in flight beside the sums
+                        const float* y = static_cast<const float*>(a.out.y0) + (size_t)(m0 + c0) * a.out.ld0 + row;
+#pragma unroll
+                        for (int j = 0; j < kChunk; ++j)
+                            if (MODE == kDenseAddF32) old[j] = c0 + j < cnt ? y[(size_t)j * a.out.ld0] : 0.f;
+                    }
                     if (plan.ksplit > 1) {
 #pragma unroll
                         for (int j = 0; j < kChunk; ++j) v[j] = __ldcg(parts + (size_t)(c0 + j) * kBlockRows);
@@ -278,25 +279,19 @@ __global__ void __launch_bounds__(kGemmThreads, 1) gemm_bf16_kernel(const __grid
                             if (row < a.rows && c0 + p < cnt) y[(size_t)p * a.out.ld0] = from_f32<bf16>(z);
                         }
                     } else if (row < a.rows) {
-                        if (a.out.bias) {
+                        if (MODE != kDenseAddF32 && a.out.bias) {
                             const float b = to_f32(a.out.bias[row]);
 #pragma unroll
                             for (int j = 0; j < kChunk; ++j) v[j] += b;
                         }
                         if (MODE == kDenseAddF32) {
                             float* y = static_cast<float*>(a.out.y0) + (size_t)(m0 + c0) * a.out.ld0 + row;
-                            float old[kChunk];
-#pragma unroll
-                            for (int j = 0; j < kChunk; ++j) old[j] = c0 + j < cnt ? y[(size_t)j * a.out.ld0] : 0.f;
 #pragma unroll
                             for (int j = 0; j < kChunk; ++j)
-                                if (c0 + j < cnt) y[(size_t)j * a.out.ld0] = old[j] + v[j];
+                                if (MODE == kDenseAddF32 && c0 + j < cnt) y[(size_t)j * a.out.ld0] = old[j] + v[j];
                         } else if (MODE == kDenseStoreF32 || (MODE == kDenseStoreMixed && row < a.out.split)) {
                             float* y = static_cast<float*>(a.out.y0) + (size_t)(m0 + c0) * a.out.ld0 + row;
-                            if (MODE == kDenseStoreF32 && a.out.act == kDenseDecay) {
-#pragma unroll
-                                for (int j = 0; j < kChunk; ++j) v[j] = expf(-expf(v[j]));
-                            }
+                            if (MODE == kDenseStoreF32 && ACT == kDenseDecay) activate<ACT>(v, a.out);
 #pragma unroll
                             for (int j = 0; j < kChunk; ++j)
                                 if (c0 + j < cnt) y[(size_t)j * a.out.ld0] = v[j];
@@ -304,7 +299,7 @@ __global__ void __launch_bounds__(kGemmThreads, 1) gemm_bf16_kernel(const __grid
                             const bool act = MODE == kDenseStoreMixed || row >= a.out.split;
                             const int ld = act ? a.out.ld1 : a.out.ld0;
                             bf16* y = (act ? static_cast<bf16*>(a.out.y1) - a.out.split : static_cast<bf16*>(a.out.y0)) + (size_t)(m0 + c0) * ld + row;
-                            if (act) activate(v, a.out);
+                            if (act) activate<ACT>(v, a.out);
 #pragma unroll
                             for (int j = 0; j < kChunk; ++j)
                                 if (c0 + j < cnt) y[(size_t)j * ld] = from_f32<bf16>(v[j]);
@@ -355,18 +350,30 @@ cudaError_t launch_bf16_t(const Launch& l, int mode, const DenseGemmArgs& a, con
     const int groups = a.group_rows ? a.groups : 1;
     if (!encode_rows(&mw, a.w, a.table ? a.rows * a.experts : a.rows, a.cols, kBlockRows) || !encode_rows(&mx, a.x, a.m + (groups - 1) * a.x_group, a.cols, BN)) return cudaErrorInvalidValue;
     const dim3 grid(std::min(plan.units, a.sm_count > 0 ? a.sm_count : 148)), block(kGemmThreads);
+    auto go = [&](auto kernel) { return launch_chained(l, kernel, grid, block, gemm_smem(BN), mw, mx, a, plan); };
     if (a.table) {
         if constexpr (BN >= 32 && BN <= 128) {
-            if (mode == kDenseStoreF32) return launch_chained(l, gemm_bf16_kernel<BN, kDenseStoreF32, true>, grid, block, gemm_smem(BN), mw, mx, a, plan);
-            if (mode == kDenseStoreGlu) return launch_chained(l, gemm_bf16_kernel<BN, kDenseStoreGlu, true>, grid, block, gemm_smem(BN), mw, mx, a, plan);
+            if (mode == kDenseStoreF32) return go(gemm_bf16_kernel<BN, kDenseStoreF32, kDenseXielu, true>);
+            if (mode == kDenseStoreGlu) return go(gemm_bf16_kernel<BN, kDenseStoreGlu, kDenseXielu, true>);
         }
         return cudaErrorInvalidValue;
     }
     switch (mode) {
-        case kDenseStoreF32: return launch_chained(l, gemm_bf16_kernel<BN, kDenseStoreF32, false>, grid, block, gemm_smem(BN), mw, mx, a, plan);
-        case kDenseAddF32: return launch_chained(l, gemm_bf16_kernel<BN, kDenseAddF32, false>, grid, block, gemm_smem(BN), mw, mx, a, plan);
-        case kDenseStoreAct: return launch_chained(l, gemm_bf16_kernel<BN, kDenseStoreAct, false>, grid, block, gemm_smem(BN), mw, mx, a, plan);
-        case kDenseStoreMixed: return launch_chained(l, gemm_bf16_kernel<BN, kDenseStoreMixed, false>, grid, block, gemm_smem(BN), mw, mx, a, plan);
+        case kDenseStoreF32: return a.out.act == kDenseDecay ? go(gemm_bf16_kernel<BN, kDenseStoreF32, kDenseDecay, false>) : go(gemm_bf16_kernel<BN, kDenseStoreF32, kDenseXielu, false>);
+        case kDenseAddF32: return go(gemm_bf16_kernel<BN, kDenseAddF32, kDenseXielu, false>);
+        case kDenseStoreAct:
+            switch (a.out.act) {
+                case kDenseXielu: return go(gemm_bf16_kernel<BN, kDenseStoreAct, kDenseXielu, false>);
+                case kDenseRelu2: return go(gemm_bf16_kernel<BN, kDenseStoreAct, kDenseRelu2, false>);
+                case kDenseTanh: return go(gemm_bf16_kernel<BN, kDenseStoreAct, kDenseTanh, false>);
+                default: return cudaErrorInvalidValue;
+            }
+        case kDenseStoreMixed:
+            switch (a.out.act) {
+                case kDenseRelu2: return go(gemm_bf16_kernel<BN, kDenseStoreMixed, kDenseRelu2, false>);
+                case kDenseTanh: return go(gemm_bf16_kernel<BN, kDenseStoreMixed, kDenseTanh, false>);
+                default: return cudaErrorInvalidValue;
+            }
         default: return cudaErrorInvalidValue;
     }
 }
@@ -503,7 +510,7 @@ cudaError_t launch_f32(const Launch& l, int mode, const DenseGemmArgs& a) {
 
 cudaError_t launch_dense_gemm(const Launch& l, DenseType type, int mode, const DenseGemmArgs& a) {
     if (a.rows <= 0 || a.cols <= 0 || a.cols % 64 || a.m <= 0 || (mode != kDenseStoreAct && mode != kDenseStoreMixed && a.out.split != a.rows)) return cudaErrorInvalidValue;
-    if ((a.group_rows && (a.group_rows % kBlockRows || a.x_group < a.m || a.groups <= 0)) || (a.table && (a.experts <= 0 || a.max_entries <= 0 || a.group_rows)) || (mode == kDenseStoreGlu && (!a.table || a.rows % kBlockRows)))
+    if ((a.group_rows && (a.group_rows % kBlockRows || a.x_group < a.m || a.groups <= 0)) || (a.table && (a.experts <= 0 || a.max_entries <= 0 || a.group_rows)) || (mode == kDenseStoreGlu && (!a.table || a.rows % kBlockRows)) || (mode == kDenseAddF32 && a.out.bias))
         return cudaErrorInvalidValue;
     if ((reinterpret_cast<uintptr_t>(a.w) | reinterpret_cast<uintptr_t>(a.x)) & 15u) return cudaErrorInvalidValue;
     return type == kDenseF32 ? launch_f32(l, mode, a) : launch_bf16(l, mode, a);

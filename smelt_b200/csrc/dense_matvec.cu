@@ -21,28 +21,32 @@ __global__ void __launch_bounds__(kThreads, 1) dense_matvec_kernel(const DenseMa
     __shared__ float s_sum[kWarps];
     const int tid = threadIdx.x;
     const int r0 = blockIdx.x * rows_per_cta, r1 = min(a.rows, r0 + rows_per_cta);
-    pdl_trigger();
-
-    auto address = [&](int row, int col) { return reinterpret_cast<const uint4*>(a.w + (size_t)row * a.cols + col); };
-    RowStream<decltype(address)> stream(address, r0, r1, a.cols, chunks, ks);
-    stream.start();
-
-    pdl_wait();
-    if (dyn_skip(a.dyn)) return;
-    float ss = 0.f;
-#pragma unroll 4
-    for (int i = tid * 4; i < chunks * kChunkCols; i += kThreads * 4) {
-        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (i < a.cols) v = *reinterpret_cast<const float4*>(a.xb && i >= a.ka ? a.xb + (i - a.ka) : a.xa + i);
-        ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
-        *reinterpret_cast<float4*>(sx + staged(i)) = v;
-    }
     float factor = 1.f;
-    if (a.norm) factor = a.gain * rsqrtf(cta_sum(ss, s_sum) / (float)a.width + a.eps);
-    else __syncthreads();
-
-    stream.run(sx, part);
-    __syncthreads();
+    const bool done = stream_rows<true>(MatrixRows{a.w, a.cols}, r0, r1, a.cols, chunks, ks, sx, part, [&] {
+        pdl_wait();
+        if (dyn_skip(a.dyn)) return false;
+        float ss = 0.f;
+#pragma unroll 4
+        for (int i = tid * 4; i < chunks * kChunkCols; i += kThreads * 4) {
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (i < a.cols) v = *reinterpret_cast<const float4*>(a.xb && i >= a.ka ? a.xb + (i - a.ka) : a.xa + i);
+            ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+            *reinterpret_cast<float4*>(sx + staged(i)) = v;
+        }
+        if (a.norm) {
+            ss = warp_sum(ss);
+            if ((tid & 31) == 0) s_sum[tid >> 5] = ss;
+        }
+        __syncthreads();
+        if (a.norm) {
+            float tot = 0.f;
+#pragma unroll
+            for (int w = 0; w < kWarps; ++w) tot += s_sum[w];
+            factor = a.gain * rsqrtf(tot / (float)a.width + a.eps);
+        }
+        return true;
+    });
+    if (!done) return;
     for (int i = tid; i < r1 - r0; i += kThreads) {
         const float v = sum_parts(part, i, ks) * factor;
         const int row = r0 + i;

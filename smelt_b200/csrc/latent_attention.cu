@@ -70,7 +70,6 @@ __global__ void __launch_bounds__(kThreads) latent_query_kernel(const LatentArgs
     extern __shared__ float sq[];  // [dp]
     __shared__ float scratch[kWarps];
     __shared__ __align__(16) float s_sum[16][kQueryCols + 4];
-    pdl_trigger();
     const int tid = threadIdx.x, r = blockIdx.z, h = blockIdx.y, grp = tid >> 4, c = blockIdx.x * kQueryCols + (tid & 15) * 8;
     const bool mine = h < a.heads && c < a.kr;
     const bf16* w = a.kv + (size_t)h * a.dp * a.kr + c;
@@ -80,6 +79,7 @@ __global__ void __launch_bounds__(kThreads) latent_query_kernel(const LatentArgs
         const int d = grp + 16 * j;
         buf[j] = mine && d < a.dp ? *reinterpret_cast<const uint4*>(w + (size_t)d * a.kr) : make_uint4(0, 0, 0, 0);
     }
+    pdl_trigger();
     pdl_wait();
     if (dyn_skip(a.dyn)) return;
     const uint32_t pos = dyn_position(a.dyn) + (uint32_t)r;
@@ -189,7 +189,6 @@ constexpr int kValueDepth = 8;  // 16-byte pieces a lane holds
 template <class TZ>
 __global__ void __launch_bounds__(kThreads) latent_values_kernel(const LatentArgs a, int rows_per_cta) {
     extern __shared__ __align__(16) float sc[];  // [kr], then the splits' weights, then [row groups][kr] sums
-    pdl_trigger();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, r = blockIdx.z, h = blockIdx.y;
     const int v0 = blockIdx.x * rows_per_cta, v1 = min(a.vp, v0 + rows_per_cta), pieces = (a.kr + 255) / 256;  // of a row
     const bf16* uv = a.kv + ((size_t)a.heads * a.dp + (size_t)h * a.vp) * a.kr;
@@ -200,6 +199,7 @@ __global__ void __launch_bounds__(kThreads) latent_values_kernel(const LatentArg
     uint4 buf[kValueDepth];
 #pragma unroll
     for (int n = 0; n < kValueDepth; ++n) buf[n] = load(n);
+    pdl_trigger();
     pdl_wait();
     if (dyn_skip(a.dyn)) return;
     // the splits' weights: exp(maximum - overall maximum) over the overall sum

@@ -38,8 +38,6 @@ __global__ void __launch_bounds__(kThreads) latent_decode_kernel(const LatentArg
     const int kd = a.kr + a.rp, pitch = pitch_of(kd), nt = a.kr / 64;
     unsigned char* sq = smem;                            // [2][kHeads] rows: high and low halves
     unsigned char* sk = smem + 2 * kHeads * pitch;       // [2][kKeys] rows
-    pdl_trigger();
-
     const uint32_t i = dyn_position(a.dyn), lo = i + 1u > a.window ? i + 1u - a.window : 0u, n = i + 1u - lo;
     uint32_t per = (n + gridDim.x - 1) / gridDim.x;
     per = (per + kKeys - 1) / kKeys * kKeys;
@@ -60,6 +58,7 @@ __global__ void __launch_bounds__(kThreads) latent_decode_kernel(const LatentArg
         }
     };
     if (tiles > 0) copy_tile(0, false, true);
+    pdl_trigger();
     pdl_wait();
     if (dyn_skip(a.dyn)) {
         cp_async_commit();

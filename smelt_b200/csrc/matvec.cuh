@@ -68,60 +68,67 @@ inline Split split_rows(int rows, int cols, int sm_count) {
 }
 constexpr size_t kMaxShared = 225 * 1024;
 
-// Rows [r0, r1) of one CTA.  address(row, col): the weights' address of a lane's eight columns.
-template <class Address>
-struct RowStream {
+// Rows [r0, r1) of one CTA: their products with the staged activation row sx go to part, [r1 - r0][ks].
+// Rows: first(row, col) is where a lane's eight columns of a row lie, after(first, r) the same of the r-th row behind it.
+// prepare() waits for the launch in front and stages the activations (ending in a barrier), false: nothing
+// is to be done; the first weights are requested ahead of it, or behind it where they depend on it (!EARLY).
+template <bool EARLY, class Rows, class Prepare>
+__device__ __forceinline__ bool stream_rows(const Rows& rows, int r0, int r1, int cols, int chunks, int ks, const float* sx, float* part, Prepare prepare) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kid = warp % ks, group = warp / ks, step = kWarps / ks * kRowsPerPass;
     struct Item { int row, chunk; };
-    const Address& address;
-    int r0, r1, cols, chunks, ks, kid, lane, step;
-    Item cur, ahead;
-    uint4 buf[kDepth][kRowsPerPass];
-
-    __device__ __forceinline__ RowStream(const Address& address, int r0, int r1, int cols, int chunks, int ks) : address(address), r0(r0), r1(r1), cols(cols), chunks(chunks), ks(ks) {
-        const int warp = threadIdx.x >> 5;
-        lane = threadIdx.x & 31;
-        kid = warp % ks;
-        step = kWarps / ks * kRowsPerPass;
-        cur = Item{r0 + warp / ks * kRowsPerPass, kid};
-        ahead = cur;
-    }
-    __device__ __forceinline__ void next(Item& it) const {
+    auto next = [&](Item& it) {
         it.chunk += ks;
         if (it.chunk >= chunks) { it.chunk = kid; it.row += step; }
-    }
-    __device__ __forceinline__ void load(const Item& it, uint4 (&dst)[kRowsPerPass]) const {
+    };
+    auto load = [&](const Item& it, uint4 (&dst)[kRowsPerPass]) {
         const int col = it.chunk * kChunkCols + lane * 8;
+        const auto p = rows.first(it.row, col);
         const bool in = col < cols;
 #pragma unroll
-        for (int r = 0; r < kRowsPerPass; ++r) dst[r] = in && it.row + r < r1 ? ld_stream(address(it.row + r, col)) : make_uint4(0, 0, 0, 0);
-    }
-    __device__ __forceinline__ void start() {
+        for (int r = 0; r < kRowsPerPass; ++r) dst[r] = in && it.row + r < r1 ? ld_stream(rows.after(p, r)) : make_uint4(0, 0, 0, 0);
+    };
+    uint4 buf[kDepth][kRowsPerPass];
+    Item cur{r0 + group * kRowsPerPass, kid}, ahead = cur;
+    if (EARLY) {
 #pragma unroll
         for (int i = 0; i < kDepth; ++i) { load(ahead, buf[i]); next(ahead); }
     }
-    // sx: the staged activation row; part: [r1 - r0][ks]
-    __device__ __forceinline__ void run(const float* sx, float* part) {
-        float acc[kRowsPerPass] = {0.f, 0.f, 0.f, 0.f};
-        while (cur.row < r1) {
+    pdl_trigger();  // behind the first requests: ahead of them it cost 0.9 us
+    if (!prepare()) return false;
+    if (!EARLY) {
 #pragma unroll
-            for (int i = 0; i < kDepth; ++i) {
-                if (cur.row >= r1) break;
-                const float4 xa = *reinterpret_cast<const float4*>(sx + cur.chunk * kChunkCols + lane * 4);
-                const float4 xb = *reinterpret_cast<const float4*>(sx + cur.chunk * kChunkCols + 128 + lane * 4);
+        for (int i = 0; i < kDepth; ++i) { load(ahead, buf[i]); next(ahead); }
+    }
+    float acc[kRowsPerPass] = {0.f, 0.f, 0.f, 0.f};
+    while (cur.row < r1) {
 #pragma unroll
-                for (int r = 0; r < kRowsPerPass; ++r) acc[r] = dot8(buf[i][r], xa, xb, acc[r]);
-                load(ahead, buf[i]);
-                next(ahead);
-                if (cur.chunk + ks >= chunks) {  // the last columns of these rows
-                    const float v = sum_four_rows(acc, lane);
-                    const int row = cur.row + (lane >> 4) * 2 + ((lane >> 3) & 1);
-                    if ((lane & 7) == 0 && row < r1) part[(size_t)(row - r0) * ks + kid] = v;
-                    acc[0] = acc[1] = acc[2] = acc[3] = 0.f;
-                }
-                next(cur);
+        for (int i = 0; i < kDepth; ++i) {
+            if (cur.row >= r1) break;
+            const float4 xa = *reinterpret_cast<const float4*>(sx + cur.chunk * kChunkCols + lane * 4);
+            const float4 xb = *reinterpret_cast<const float4*>(sx + cur.chunk * kChunkCols + 128 + lane * 4);
+#pragma unroll
+            for (int r = 0; r < kRowsPerPass; ++r) acc[r] = dot8(buf[i][r], xa, xb, acc[r]);
+            load(ahead, buf[i]);
+            next(ahead);
+            if (cur.chunk + ks >= chunks) {  // the last columns of these rows
+                const float v = sum_four_rows(acc, lane);
+                const int row = cur.row + (lane >> 4) * 2 + ((lane >> 3) & 1);
+                if ((lane & 7) == 0 && row < r1) part[(size_t)(row - r0) * ks + kid] = v;
+                acc[0] = acc[1] = acc[2] = acc[3] = 0.f;
             }
+            next(cur);
         }
     }
+    __syncthreads();
+    return true;
+}
+
+// Rows of one matrix.
+struct MatrixRows {
+    const bf16* w;
+    int cols;
+    __device__ __forceinline__ const uint4* first(int row, int col) const { return reinterpret_cast<const uint4*>(w + (size_t)row * cols + col); }
+    __device__ __forceinline__ const uint4* after(const uint4* p, int r) const { return p + (size_t)r * (cols / 8); }
 };
 
 __device__ __forceinline__ float sum_parts(const float* part, int i, int ks) {

@@ -51,6 +51,38 @@ __device__ __forceinline__ void choose_experts(float* sl, int experts, int top, 
     __syncwarp();
 }
 
+// Rows of one matrix, or of the chosen experts' matrices (of rows x cols each): one behind the other, or side by side.
+template <int IN>
+struct Rows : MatrixRows {
+    __device__ __forceinline__ Rows(const StackMatvecArgs& a, const int*) : MatrixRows{a.w, a.cols} {}
+};
+template <>
+struct Rows<kInExpertsIn> {
+    const bf16* w;
+    int rows, cols;
+    const int* expert;
+    struct Pairs { const uint4 *low, *high; };
+    __device__ __forceinline__ Rows(const StackMatvecArgs& a, const int* expert) : w(a.w), rows(a.rows), cols(a.cols), expert(expert) {}
+    __device__ __forceinline__ const uint4* at(int row, int col) const {
+        const int n = min(row / rows, kMaxTop - 1);  // rows past the last expert's are not read
+        return reinterpret_cast<const uint4*>(w + ((size_t)expert[n] * rows + (row - n * rows)) * cols + col);
+    }
+    __device__ __forceinline__ Pairs first(int row, int col) const { return {at(row, col), at(row + 2, col)}; }  // an even number of rows an expert: a pair is never divided
+    __device__ __forceinline__ const uint4* after(const Pairs& p, int r) const { return (r < 2 ? p.low : p.high) + (r & 1) * (cols / 8); }
+};
+template <>
+struct Rows<kInExpertsOut> {
+    const bf16* w;
+    int rows, cols;
+    const int* expert;
+    __device__ __forceinline__ Rows(const StackMatvecArgs& a, const int* expert) : w(a.w), rows(a.rows), cols(a.cols), expert(expert) {}
+    __device__ __forceinline__ const uint4* first(int row, int col) const {
+        const int n = min(col / cols, kMaxTop - 1);  // columns past the last expert's are not read
+        return reinterpret_cast<const uint4*>(w + ((size_t)expert[n] * rows + row) * cols + (col - n * cols));
+    }
+    __device__ __forceinline__ const uint4* after(const uint4* p, int r) const { return p + (size_t)r * (cols / 8); }
+};
+
 template <int IN>
 __global__ void __launch_bounds__(kThreads, 1) stack_matvec_kernel(const StackMatvecArgs a, int rows_per_cta, int ks) {
     extern __shared__ __align__(16) float smem[];
@@ -69,115 +101,99 @@ __global__ void __launch_bounds__(kThreads, 1) stack_matvec_kernel(const StackMa
         r0 = group * a.group_rows + ((int)blockIdx.x - group * per_group) * rows_per_cta;
         r1 = min(group == kMixes - 1 ? a.rows : (group + 1) * a.group_rows, r0 + rows_per_cta);
     }
-    pdl_trigger();
-
-    auto address = [&](int row, int col) {
-        if (IN == kInExpertsIn) {
-            const int n = row / a.rows;
-            return reinterpret_cast<const uint4*>(a.w + ((size_t)s_expert[n] * a.rows + (row - n * a.rows)) * a.cols + col);
-        }
-        if (IN == kInExpertsOut) {
-            const int n = col / a.cols;
-            return reinterpret_cast<const uint4*>(a.w + ((size_t)s_expert[n] * a.rows + row) * a.cols + (col - n * a.cols));
-        }
-        return reinterpret_cast<const uint4*>(a.w + (size_t)row * a.cols + col);
-    };
-    RowStream<decltype(address)> stream(address, r0, r1, cols, chunks, ks);
-    if (!kSelect) stream.start();
-
-    pdl_wait();
-    if (dyn_skip(a.dyn)) return;
-    const int staged_cols = chunks * kChunkCols;
     float factor = 1.f;
-    if (IN == kInExpertsIn) {
-        float* sl = part + (size_t)rows_per_cta * ks;  // [experts]
-        for (int i = tid; i < a.experts; i += kThreads) sl[i] = a.logits[i];
-        __syncthreads();
-        if (tid < 32) {
-            choose_experts(sl, a.experts, a.top, s_expert, s_weight, tid);
-            if (blockIdx.x == 0)
-                for (int n = tid; n < a.top; n += 32) a.chosen[n] = make_int2(s_expert[n], __float_as_int(s_weight[n]));
-        }
-    } else if (IN == kInExpertsOut) {
-        if (tid < a.top) s_expert[tid] = a.chosen[tid].x;
-    }
-    if (IN == kInPlain || kSelect) {
-#pragma unroll 4
-        for (int i = tid * 4; i < staged_cols; i += kThreads * 4)
-            *reinterpret_cast<float4*>(sx + staged(i)) = i < cols ? *reinterpret_cast<const float4*>(a.x + i) : make_float4(0.f, 0.f, 0.f, 0.f);
-        __syncthreads();
-    } else if (IN == kInNorm) {
-        float ss = 0.f;
-#pragma unroll 4
-        for (int i = tid * 4; i < staged_cols; i += kThreads * 4) {
-            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (i < cols) {
-                v = *reinterpret_cast<const float4*>(a.x + i);
-                ss = sumsq4(v, ss);
-                const float4 w = ld_bf16x4(a.norm_w + i);
-                v = make_float4(v.x * w.x, v.y * w.y, v.z * w.z, v.w * w.w);
+    const bool done = stream_rows<!kSelect>(Rows<IN>(a, s_expert), r0, r1, cols, chunks, ks, sx, part, [&] {
+        pdl_wait();
+        if (dyn_skip(a.dyn)) return false;
+        const int staged_cols = chunks * kChunkCols;
+        if (IN == kInExpertsIn) {
+            float* sl = part + (size_t)rows_per_cta * ks;  // [experts]
+            for (int i = tid; i < a.experts; i += kThreads) sl[i] = a.logits[i];
+            __syncthreads();
+            if (tid < 32) {
+                choose_experts(sl, a.experts, a.top, s_expert, s_weight, tid);
+                if (blockIdx.x == 0)
+                    for (int n = tid; n < a.top; n += 32) a.chosen[n] = make_int2(s_expert[n], __float_as_int(s_weight[n]));
             }
-            *reinterpret_cast<float4*>(sx + staged(i)) = v;
+        } else if (IN == kInExpertsOut) {
+            if (tid < a.top) s_expert[tid] = a.chosen[tid].x;
         }
-        factor = rsqrtf(cta_sum(ss, s_sum[0]) / (float)a.width + a.eps);
-    } else {
-        float fy = 0.f;
-        if (a.y) {
+        if (IN == kInPlain || kSelect) {
+#pragma unroll 4
+            for (int i = tid * 4; i < staged_cols; i += kThreads * 4)
+                *reinterpret_cast<float4*>(sx + staged(i)) = i < cols ? *reinterpret_cast<const float4*>(a.x + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+            __syncthreads();
+        } else if (IN == kInNorm) {
             float ss = 0.f;
 #pragma unroll 4
-            for (int i = tid * 4; i < cols; i += kThreads * 4) {
-                const float4 v = *reinterpret_cast<const float4*>(a.y + i);
-                ss = sumsq4(v, ss);
-                *reinterpret_cast<float4*>(sx + staged(i)) = v;  // read again by this thread only
-            }
-            fy = rsqrtf(cta_sum(ss, s_sum[0]) / (float)a.width + a.eps);
-        }
-        float ss = 0.f;
-#pragma unroll 4
-        for (int i = tid * 4; i < staged_cols; i += kThreads * 4) {
-            float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (i < cols) {
-                s = *reinterpret_cast<const float4*>(a.x + i);
-                if (a.y) {
-                    const float4 y = *reinterpret_cast<const float4*>(sx + staged(i)), w = ld_bf16x4(a.post_w + i);
-                    s.x = fmaf(y.x * fy, 1.f + w.x, s.x);
-                    s.y = fmaf(y.y * fy, 1.f + w.y, s.y);
-                    s.z = fmaf(y.z * fy, 1.f + w.z, s.z);
-                    s.w = fmaf(y.w * fy, 1.f + w.w, s.w);
-                    if (blockIdx.x == 0 && a.x_out) *reinterpret_cast<float4*>(a.x_out + i) = s;
+            for (int i = tid * 4; i < staged_cols; i += kThreads * 4) {
+                float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (i < cols) {
+                    v = *reinterpret_cast<const float4*>(a.x + i);
+                    ss = sumsq4(v, ss);
+                    const float4 w = ld_bf16x4(a.norm_w + i);
+                    v = make_float4(v.x * w.x, v.y * w.y, v.z * w.z, v.w * w.w);
                 }
-                ss = sumsq4(s, ss);
-                const float4 w = ld_bf16x4(a.norm_w + i);
-                s = make_float4(s.x * (1.f + w.x), s.y * (1.f + w.y), s.z * (1.f + w.z), s.w * (1.f + w.w));
+                *reinterpret_cast<float4*>(sx + staged(i)) = v;
             }
-            *reinterpret_cast<float4*>(sx + staged(i)) = s;
-        }
-        factor = rsqrtf(cta_sum(ss, s_sum[1]) / (float)a.width + a.eps);
-        const bool store_h = a.h_out && blockIdx.x == 0;
-        if (IN == kInShift || store_h) {
-            const bool has_before = IN == kInShift && dyn_position(a.dyn) != 0u;
-            const bf16* mu = IN == kInShift ? a.mu + (size_t)group * a.cols : nullptr;
+            factor = rsqrtf(cta_sum(ss, s_sum[0]) / (float)a.width + a.eps);
+        } else {
+            float fy = 0.f;
+            if (a.y) {
+                float ss = 0.f;
 #pragma unroll 4
-            for (int i = tid * 4; i < cols; i += kThreads * 4) {
-                float4* at = reinterpret_cast<float4*>(sx + staged(i));
-                float4 h = *at;
-                h = make_float4(h.x * factor, h.y * factor, h.z * factor, h.w * factor);
-                if (store_h) *reinterpret_cast<float4*>(a.h_out + i) = h;
-                if (IN == kInShift) {
-                    const float4 b = has_before ? *reinterpret_cast<const float4*>(a.before + i) : make_float4(0.f, 0.f, 0.f, 0.f), t = ld_bf16x4(mu + i);
-                    *at = make_float4(fmaf(b.x - h.x, t.x, h.x), fmaf(b.y - h.y, t.y, h.y), fmaf(b.z - h.z, t.z, h.z), fmaf(b.w - h.w, t.w, h.w));
+                for (int i = tid * 4; i < cols; i += kThreads * 4) {
+                    const float4 v = *reinterpret_cast<const float4*>(a.y + i);
+                    ss = sumsq4(v, ss);
+                    *reinterpret_cast<float4*>(sx + staged(i)) = v;  // read again by this thread only
+                }
+                fy = rsqrtf(cta_sum(ss, s_sum[0]) / (float)a.width + a.eps);
+            }
+            float ss = 0.f;
+#pragma unroll 4
+            for (int i = tid * 4; i < staged_cols; i += kThreads * 4) {
+                float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (i < cols) {
+                    s = *reinterpret_cast<const float4*>(a.x + i);
+                    if (a.y) {
+                        const float4 y = *reinterpret_cast<const float4*>(sx + staged(i)), w = ld_bf16x4(a.post_w + i);
+                        s.x = fmaf(y.x * fy, 1.f + w.x, s.x);
+                        s.y = fmaf(y.y * fy, 1.f + w.y, s.y);
+                        s.z = fmaf(y.z * fy, 1.f + w.z, s.z);
+                        s.w = fmaf(y.w * fy, 1.f + w.w, s.w);
+                        if (blockIdx.x == 0 && a.x_out) *reinterpret_cast<float4*>(a.x_out + i) = s;
+                    }
+                    ss = sumsq4(s, ss);
+                    const float4 w = ld_bf16x4(a.norm_w + i);
+                    s = make_float4(s.x * (1.f + w.x), s.y * (1.f + w.y), s.z * (1.f + w.z), s.w * (1.f + w.w));
+                }
+                *reinterpret_cast<float4*>(sx + staged(i)) = s;
+            }
+            factor = rsqrtf(cta_sum(ss, s_sum[1]) / (float)a.width + a.eps);
+            const bool store_h = a.h_out && blockIdx.x == 0;
+            if (IN == kInShift || store_h) {
+                const bool has_before = IN == kInShift && dyn_position(a.dyn) != 0u;
+                const bf16* mu = IN == kInShift ? a.mu + (size_t)group * a.cols : nullptr;
+#pragma unroll 4
+                for (int i = tid * 4; i < cols; i += kThreads * 4) {
+                    float4* at = reinterpret_cast<float4*>(sx + staged(i));
+                    float4 h = *at;
+                    h = make_float4(h.x * factor, h.y * factor, h.z * factor, h.w * factor);
+                    if (store_h) *reinterpret_cast<float4*>(a.h_out + i) = h;
+                    if (IN == kInShift) {
+                        const float4 b = has_before ? *reinterpret_cast<const float4*>(a.before + i) : make_float4(0.f, 0.f, 0.f, 0.f), t = ld_bf16x4(mu + i);
+                        *at = make_float4(fmaf(b.x - h.x, t.x, h.x), fmaf(b.y - h.y, t.y, h.y), fmaf(b.z - h.z, t.z, h.z), fmaf(b.w - h.w, t.w, h.w));
+                    }
                 }
             }
+            if (IN == kInShift) {
+                factor = 1.f;
+                __syncthreads();
+            }
         }
-        if (IN == kInShift) {
-            factor = 1.f;
-            __syncthreads();
-        }
-    }
-
-    if (kSelect) stream.start();
-    stream.run(sx, part);
-    __syncthreads();
+        return true;
+    });
+    if (!done) return;
     if (IN == kInExpertsIn) {  // pairs of rows: gate, up
         for (int i = tid; i < (r1 - r0) / 2; i += kThreads)
             a.out[r0 / 2 + i] = clamped_glu(sum_parts(part, 2 * i, ks), sum_parts(part, 2 * i + 1, ks), a.limit) * s_weight[(r0 + 2 * i) / a.rows];

@@ -37,7 +37,6 @@ template <int D, int VD, int NH>
 __global__ void __launch_bounds__(kAttnThreads) window_decode_kernel(const WindowArgs a, const CapWeight cw, int head_groups) {
     constexpr int NU = ring_units_of<D, VD>(), UB = unit_bytes<D, VD>(), KJ = D / 32, VC = VD / 64, HN = NH * 8;
     extern __shared__ __align__(16) unsigned char smem[];
-    pdl_trigger();
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
     const int splits = gridDim.x, split = blockIdx.x, kvh = blockIdx.y / head_groups, hgroup = blockIdx.y % head_groups;
     const int ratio = a.heads / a.kv_heads, head0 = kvh * ratio + hgroup * HN, heads = min(HN, ratio - hgroup * HN);
@@ -91,6 +90,7 @@ __global__ void __launch_bounds__(kAttnThreads) window_decode_kernel(const Windo
         if (kt < k_end && kt + 16 > n - 1u) break;  // holds the new token's row
         issue_unit(issued);
     }
+    pdl_trigger();
     pdl_wait();
     if (dyn_skip(a.dyn)) {
         cp_async_wait<0>();

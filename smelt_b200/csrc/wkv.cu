@@ -41,7 +41,6 @@ __global__ void __launch_bounds__(kThreads) wkv_decode_kernel(const WkvArgs a, i
     float* so = st + a.rank;                                                  // [groups][D]
     float* ss = smem + ((4 * D + a.rank + groups * D + 3) & ~3);              // [D][D] where it fits
     float* state = a.state + (size_t)h * D * D;
-    pdl_trigger();
     if (state_smem) {  // the last token's state: only this kernel writes it
         for (int i = tid; i < D * D / 4; i += kThreads) cp_async16(ss + 4 * i, state + 4 * i);
         cp_async_commit();
@@ -56,6 +55,7 @@ __global__ void __launch_bounds__(kThreads) wkv_decode_kernel(const WkvArgs a, i
     uint4 held[kHeld];
 #pragma unroll
     for (int n = 0; n < kHeld; ++n) held[n] = n < passes * pieces ? w2_piece(n) : make_uint4(0, 0, 0, 0);
+    pdl_trigger();
     pdl_wait();
     if (dyn_skip(a.dyn)) {
         cp_async_wait<0>();
