@@ -5,8 +5,8 @@
 // A CTA owns a contiguous range of rows; its sixteen warps form 16 / ks row groups of ks warps that
 // split the columns.  A warp's work is a sequence of items of four rows x 256 columns, so that every
 // activation value read from shared memory feeds four weights; kDepth items are in flight in
-// registers (256 bytes a lane), across the end of a group of rows and, when the caller starts the
-// stream early, across its wait for the launch in front.  Partial sums go to shared memory, [row of
+// registers (256 bytes a lane), across the end of a group of rows and, where the weights do not
+// depend on it, across the wait for the launch in front.  Partial sums go to shared memory, [row of
 // the CTA][ks], and are added in warp order by the caller.
 #pragma once
 #include "dense.h"
@@ -53,7 +53,7 @@ __device__ __forceinline__ int staged(int i) {
 // ks and the rows a CTA takes: one CTA per SM with an equal share, at least what keeps its row groups busy.
 struct Split {
     int chunks, ks, rows_per_cta;
-    size_t smem(int extra_rows = 0) const { return (size_t)chunks * kChunkCols * sizeof(float) + (size_t)(rows_per_cta + extra_rows) * ks * sizeof(float); }
+    size_t smem() const { return (size_t)chunks * kChunkCols * sizeof(float) + (size_t)rows_per_cta * ks * sizeof(float); }
 };
 inline Split split_rows(int rows, int cols, int sm_count) {
     const int sm = sm_count > 0 ? sm_count : 148;
